@@ -1,9 +1,10 @@
 // stack.cu — the layer-stack model family on the B200 engine: configuration (config.json), weights (model.safetensors),
 // per-sequence state (attention cache + recurrent state), the step function for prompt portions and single tokens, and
-// the registry of designs and mixers. Kernels: stack_kernels.cuh, stack_kernels_mix.cuh, stack_kernels_hyper.cuh. C-ABI dispatch: engine.cu.
+// the registry of designs and mixers. Kernels: stack_kernels.cuh, stack_kernels_mix.cuh,
+// stack_kernels_hyper.cuh, stack_kernels_scan.cuh. C-ABI dispatch: engine.cu.
 //
 // A design is a name in config.json ("architecture") mapped to a builder that turns the configuration into a list of
-// LayerSpec; a mixer is a name ("type") mapped to a loader of its tensors and a forward routine. Four designs are registered:
+// LayerSpec; a mixer is a name ("type") mapped to a loader of its tensors and a forward routine. Five designs are registered:
 //   Matulorn   sequential sub-layers with grouped norms before and after each; mixers minGRU | latent attention (rotated
 //              part, window, sink) | gated delta rule; clamped gated feed-forward
 //   Dopilorn   both sub-layers read the same residual (x += mixer(n1 x) + ff(n2 x)) behind a causal convolution of their
@@ -21,12 +22,18 @@
 //              values (rotation of neighbouring pairs); both may mix their values with the first such layer's | latent
 //              attention (causal, gated entry by entry). Routed mixture: sigmoid scores, experts run on the weighted input,
 //              an ungated shared unit
+//   Kogerax    sub-layers read the residual itself and are normed on the way out (zero-centred weights), scaled, and added; scaled
+//              embedding. Mixers: parallel (soft-max attention over grouped heads with unit queries and keys and a sliding
+//              window beside a selective scan, each normed, averaged) | mLSTM | state-space duality (mamba2). Feed-forward: gelu
+//              unit | routed mixture (soft-max over experts and identity outputs, a correction on the choice, normalised
+//              weights, clamped units, a gated shared unit)
 // A model is executed as a list of layer RUNS: (layer, state slot), one per layer unless the design repeats some.
 #include "stack.hpp"
 #include "safetensors.hpp"
 #include "stack_kernels.cuh"
 #include "stack_kernels_mix.cuh"
 #include "stack_kernels_hyper.cuh"
+#include "stack_kernels_scan.cuh"
 
 #include <algorithm>
 #include <cmath>
@@ -44,8 +51,8 @@ using namespace stk;
 
 namespace {
 
-enum MixerKind { MIX_MINGRU = 0, MIX_LATENT, MIX_DELTA, MIX_GDELTA, MIX_DIFFATTN, MIX_RETENTION, MIX_SIGATTN, MIX_PAIR, MIX_GQATTN };
-enum BlockKind { BLOCK_SEQUENTIAL = 0, BLOCK_PARALLEL, BLOCK_PRENORM, BLOCK_HYPER };
+enum MixerKind { MIX_MINGRU = 0, MIX_LATENT, MIX_DELTA, MIX_GDELTA, MIX_DIFFATTN, MIX_RETENTION, MIX_SIGATTN, MIX_PAIR, MIX_GQATTN, MIX_SELSCAN, MIX_MLSTM, MIX_SSD };
+enum BlockKind { BLOCK_SEQUENTIAL = 0, BLOCK_PARALLEL, BLOCK_PRENORM, BLOCK_HYPER, BLOCK_POSTNORM };
 enum FfKind { FF_GLU = 0, FF_POLY, FF_MOE };
 constexpr int CHUNK_MAX = 512;          // tokens per pass of a prompt portion (longer steps run as several passes)
 constexpr float GLU_ALPHA = 1.702f;     // the feed-forward's sigmoid slope: fixed by the design
@@ -89,10 +96,16 @@ struct LayerSpec {
     // feed-forward
     int ff = 0, ff_kind = FF_GLU;
     float limit = 0.f;
+    int act_kind = GLU_SIGMOID;          // gated units: GLU_*
+    float act_alpha = GLU_ALPHA, act_shift = 1.f;      // GLU_SIGMOID: the sigmoid's slope and what is added to the up half
     DMat gateup, down;                   // FF_POLY: gateup is the plain up-projection; FF_MOE: the shared unit (ff = 0: none)
     float * act = nullptr;               // FF_POLY: the four coefficients
     // FF_MOE: routed mixture of gated units. e_gateup [n_exp][2 e_ff][E] (gate / up interleaved), e_down [n_exp][E][e_ff]
     int n_exp = 0, top = 0, n_groups = 1, keep_groups = 1, e_ff = 0;
+    int n_ident = 0;                     // router outputs n_exp .. n_exp + n_ident - 1 are identity experts: the input itself, no matrices
+    float e_limit = INFINITY;            // clamp of the experts' units (`limit`: the shared unit's)
+    float * corr = nullptr;              // added to the scores when experts are chosen, not when they are weighed
+    bool norm_w = false;                 // the chosen scores are divided by their sum
     float r_scale = 1.f;
     int route_fn = 0;                    // 0: soft-max over the experts; 1: sigmoid of each logit
     bool scale_input = false;            // the choice's weight multiplies the expert's input instead of its output
@@ -118,6 +131,16 @@ struct LayerSpec {
     float * r1 = nullptr, * r2 = nullptr;
     int vmode = 0;                       // GQA_V_*: values left for later layers / mixed with the first mixing layer's
     float vlambda = 0.f;
+    bool unit_qk = false;                // q and k over their root mean square, no weight
+    // selective scan: proj = x | z; wx maps the convolved x to [ step latent | B | C ]; wdt maps the latent to `inner` step sizes (bias)
+    int inner = 0, state = 0, dt_rank = 0;
+    DMat wx, wdt;
+    float * bconv = nullptr, * skip = nullptr;       // convolution bias; factor on the convolved input added to the read-out
+    // state-space duality: proj = z | x | B | C | dt; D = state entries, KH = groups; A_log, dt_bias, dnorm, wconv above
+    int norm_parts = 1;
+    // mLSTM: proj = q | k | v | output gate | input gate | forget gate (biases on the last two); a head keeps [D][V] and n [D]
+    float gate_cap = 0.f;
+    size_t head_stride = 0;
     // hyper-connections (BLOCK_HYPER): the weights of both sub-layers, and norm weights that are one number
     HcW hc[2];
     float g1 = 1.f, g2 = 1.f;
@@ -159,8 +182,11 @@ struct StackModel {
     bool rope_adjacent = false;           // the design rotates neighbouring pairs
     int vfirst_width = 0, vfirst_heads = 0;   // key/value heads x vdim, and key/value heads, of the first value-mixing layer (0: none so far)
     int max_slots = 0, max_eff = 0, max_exp = 0;      // routed mixtures: choices per token, expert width, experts
-    size_t max_ret_state = 0;             // retention: the largest heads x dim x vdim
-    int max_ret_dim = 0;
+    size_t max_scan_state = 0;            // outer-product recurrences: the largest matrix state of a layer
+    int max_scan_dim = 0, max_scan_heads = 0;
+    float residual_mult = 1.f, embed_scale = 1.f;     // BLOCK_POSTNORM: factor on a sub-layer's normed output; on the embedding row
+    bool unit_qk = false;                 // the design's attention has unit queries and keys
+    const char * pair_default[2] = { "sigmoid_attention", "retention" };      // mixers of a pair whose branches name none
     DMat loop_in;                         // repeated span: [E][2 E]
     float * loop_step = nullptr;          // [times][E]
     std::vector<LayerSpec> layers;
@@ -211,7 +237,8 @@ struct StackCtx {
     size_t att_scores_floats = 0;
     std::vector<float *> cache_allocs;    // the caches with their zero margins (caches[] point behind the front margin)
     float * att_part = nullptr, * att_ml = nullptr;   // key-slice partials of the latent attention (decode)
-    float * ret_sb = nullptr;             // retention, long portions: per-chunk states [heads][chunks][dim][vdim]
+    float * scan_sb = nullptr, * scan_ac = nullptr;      // outer-product recurrences, long portions: per-chunk states [heads][chunks][state], decays [heads][chunks]
+    float * den = nullptr;                // mLSTM: n . q [cap][heads]
     float * keep = nullptr;               // depth average: [layers + 1][cap][E] results of this pass's tokens
     float * Xp = nullptr, * Ap = nullptr, * Yk = nullptr, * r_wt = nullptr, * r_sg = nullptr;      // routed mixture: rows by slot, weights, shared gate
     int32_t * r_sel = nullptr, * r_slot = nullptr, * r_src = nullptr, * r_seg = nullptr;
@@ -458,7 +485,9 @@ void load_diffattn(StackModel & m, LayerSpec & L, const Json & mx, const safeten
     m.maxQK = std::max(m.maxQK, nq); m.maxOL = std::max(m.maxOL, H * V);      // prompt portions: regrouped queries, per-group outputs
 }
 
-// plain rotary frequencies f_i = base^(-2i/dims) of a mixer's "rot" object (absent: no rotation)
+// rotary frequencies f_i = base^(-2i/dims) of a mixer's "rot" object (absent: no rotation). With "scaling" {factor, low, high, original}
+// a frequency of wavelength l = 2 pi / f stays when original / l > high, is divided by `factor` when original / l < low, and is blended
+// linearly in original / l in between
 void load_rot(StackModel & m, LayerSpec & L, const Json & mx, int D) {
     L.rope_dims = 0; L.rope_mag = 1.f;
     std::vector<float> freq(1, 0.f);
@@ -468,9 +497,27 @@ void load_rot(StackModel & m, LayerSpec & L, const Json & mx, int D) {
         if (dims < 0 || dims > D || dims % 2) throw std::runtime_error("config: rot.dims must be even and at most dim");
         const double base = rot.number("base");
         freq.assign((size_t) std::max(dims / 2, 1), 0.f);
-        for (int i = 0; i < dims / 2; i++) freq[(size_t) i] = (float) std::pow(base, -2.0 * i / dims);
+        const bool scaled = rot.has("scaling");
+        double factor = 1.0, low = 0, high = 0, orig = 0;
+        if (scaled) { const Json & sc = rot.at("scaling"); factor = sc.number("factor"); low = sc.number("low"); high = sc.number("high"); orig = sc.number("original"); }
+        for (int i = 0; i < dims / 2; i++) {
+            double f = std::pow(base, -2.0 * i / dims);
+            if (scaled) {
+                const double wave = 2.0 * M_PI / f;
+                if (wave > orig / low) f /= factor;
+                else if (!(wave < orig / high)) { const double s = (orig / wave - low) / (high - low); f = (1.0 - s) * f / factor + s * f; }
+            }
+            freq[(size_t) i] = (float) f;
+        }
     }
     L.rope_freq = up_f32(m, freq);
+}
+
+// bookkeeping of a matrix state [heads][head_stride] walked by the outer-product recurrence
+void note_outer_state(StackModel & m, LayerSpec & L, int heads, int dim, size_t head_stride) {
+    L.head_stride = head_stride;
+    m.max_scan_state = std::max(m.max_scan_state, (size_t) heads * head_stride);
+    m.max_scan_dim = std::max(m.max_scan_dim, dim); m.max_scan_heads = std::max(m.max_scan_heads, heads);
 }
 
 // retention: '<prefix>{q,k,v,g,o}'; decay per head from the configuration
@@ -493,7 +540,7 @@ void load_retention(StackModel & m, LayerSpec & L, const Json & mx, const safete
     L.o = up_mat(m, sf.read_f32(p + "o", {E, H * V}), E, H * V, nullptr);
     L.n_rec = (size_t) H * D * V;
     m.maxP = std::max(m.maxP, L.proj.N); m.maxA = std::max(m.maxA, H * V);
-    m.max_ret_state = std::max(m.max_ret_state, L.n_rec); m.max_ret_dim = std::max(m.max_ret_dim, D);
+    note_outer_state(m, L, H, D, (size_t) D * V);
 }
 
 // sigmoid attention: '<prefix>{q,k,v,q.norm,k.norm,pb,o}'; slopes 2^(-8 (h + 1) / H) are fixed by the mechanism
@@ -545,6 +592,7 @@ void load_gqattn(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
     }
     load_rot(m, L, mx, D);
     L.rope_adjacent = m.rope_adjacent;
+    L.unit_qk = m.unit_qk;
     std::vector<float> W = sf.read_f32(p + "q", {H * D, E});
     append(W, sf.read_f32(p + "k", {G * D, E}));
     append(W, sf.read_f32(p + "v", {G * V, E}));
@@ -572,6 +620,73 @@ void load_gqattn(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
 void load_gqattn_chunks(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) { load_gqattn(m, L, mx, sf, p, MASK_CHUNK); }
 void load_gqattn_window(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) { load_gqattn(m, L, mx, sf, p, MASK_WINDOW); }
 
+// selective scan: '<prefix>{in,conv,conv.b,x,dt,dt.b,A_log,D,o}'
+void load_selscan(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) {
+    const int E = m.E, n = L.inner = need_int(mx, "inner"), N = L.state = need_int(mx, "state"), R = L.dt_rank = need_int(mx, "dt_rank");
+    const int taps = L.taps = need_int(mx, "conv");
+    if (N > 256) throw std::runtime_error("selective scan: more than 256 state entries per channel are not supported");
+    if (taps > 64) throw std::runtime_error("config: conv taps out of range");
+    if (R > 8192) throw std::runtime_error("selective scan: dt_rank above 8192 is not supported");
+    L.proj = up_mat(m, sf.read_f32(p + "in", {2 * n, E}), 2 * n, E, nullptr);
+    L.wconv = up_f32(m, sf.read_f32(p + "conv", {n, taps}));
+    L.bconv = up_f32(m, sf.read_f32(p + "conv.b", {n}));
+    L.wx = up_mat(m, sf.read_f32(p + "x", {R + 2 * N, n}), R + 2 * N, n, nullptr);
+    const std::vector<float> db = sf.read_f32(p + "dt.b", {n});
+    L.wdt = up_mat(m, sf.read_f32(p + "dt", {n, R}), n, R, &db);
+    L.A_log = up_f32(m, sf.read_f32(p + "A_log", {n, N}));
+    L.skip = up_f32(m, sf.read_f32(p + "D", {n}));
+    L.o = up_mat(m, sf.read_f32(p + "o", {E, n}), E, n, nullptr);
+    m.weight_bytes += (int64_t) n * (N + taps + 2) * 4;
+    L.n_rec = (size_t) n * N + (size_t) (taps - 1) * n;
+    m.maxP = std::max(m.maxP, 2 * n); m.maxA = std::max(m.maxA, n); m.maxCV = std::max(m.maxCV, n);
+    m.maxBG = std::max(m.maxBG, (R + 2 * N + 3) / 4 * 4);
+}
+
+// mLSTM: '<prefix>{q,k,v,g,i,i.b,f,f.b,norm,o}'
+void load_mlstm(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) {
+    const int E = m.E, H = L.H = need_int(mx, "heads"), D = L.D = need_int(mx, "dim"), V = L.V = need_int(mx, "vdim");
+    if (D > 256) throw std::runtime_error("mLSTM: dim above 256 is not supported by the recurrence kernel");
+    L.gate_cap = (float) mx.number("gate_cap");
+    if (!(L.gate_cap > 0.f)) throw std::runtime_error("config: gate_cap must be positive");
+    std::vector<float> W = sf.read_f32(p + "q", {H * D, E}), b((size_t) 2 * H * D + 2 * H * V, 0.f);
+    append(W, sf.read_f32(p + "k", {H * D, E}));
+    append(W, sf.read_f32(p + "v", {H * V, E}));
+    append(W, sf.read_f32(p + "g", {H * V, E}));
+    append(W, sf.read_f32(p + "i", {H, E})); append(b, sf.read_f32(p + "i.b", {H}));
+    append(W, sf.read_f32(p + "f", {H, E})); append(b, sf.read_f32(p + "f.b", {H}));
+    L.proj = up_mat(m, W, 2 * H * D + 2 * H * V + 2 * H, E, &b);
+    L.dnorm = up_f32(m, sf.read_f32(p + "norm", {H * V}));
+    L.o = up_mat(m, sf.read_f32(p + "o", {E, H * V}), E, H * V, nullptr);
+    note_outer_state(m, L, H, D, (size_t) D * V + (D + 3) / 4 * 4);        // the matrix, then the normaliser
+    L.n_rec = (size_t) H * L.head_stride + H;                               // then the running maxima
+    m.maxP = std::max(m.maxP, L.proj.N); m.maxA = std::max(m.maxA, H * V);
+    m.maxBG = std::max(m.maxBG, 3 * H);
+}
+
+// state-space duality: '<prefix>{in,conv,conv.b,dt_bias,A_log,D,norm,o}'
+void load_ssd(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) {
+    const int E = m.E, H = L.H = need_int(mx, "heads"), V = L.V = need_int(mx, "vdim"), N = L.D = need_int(mx, "state");
+    const int G = L.KH = (int) mx.integer("groups", 1), taps = L.taps = need_int(mx, "conv"), inner = L.inner = H * V, C = inner + 2 * G * N;
+    L.norm_parts = (int) mx.integer("norm_groups", 1);
+    if (G < 1 || H % G) throw std::runtime_error("config: mamba2 heads must be a multiple of groups");
+    if (L.norm_parts < 1 || inner % L.norm_parts) throw std::runtime_error("config: heads x vdim must be a multiple of norm_groups");
+    if (N > 256) throw std::runtime_error("state-space duality: state above 256 is not supported by the recurrence kernel");
+    if (taps > 64) throw std::runtime_error("config: conv taps out of range");
+    L.proj = up_mat(m, sf.read_f32(p + "in", {inner + C + H, E}), inner + C + H, E, nullptr);
+    L.wconv = up_f32(m, sf.read_f32(p + "conv", {C, taps}));
+    L.bconv = up_f32(m, sf.read_f32(p + "conv.b", {C}));
+    L.dt_bias = up_f32(m, sf.read_f32(p + "dt_bias", {H}));
+    L.A_log = up_f32(m, sf.read_f32(p + "A_log", {H}));
+    L.skip = up_f32(m, sf.read_f32(p + "D", {H}));
+    L.dnorm = up_f32(m, sf.read_f32(p + "norm", {inner}));
+    L.o = up_mat(m, sf.read_f32(p + "o", {E, inner}), E, inner, nullptr);
+    note_outer_state(m, L, H, N, (size_t) N * V);
+    L.n_rec = ((size_t) H * N * V + 3) / 4 * 4 + (size_t) (taps - 1) * C;
+    m.weight_bytes += (int64_t) C * (taps + 1) * 4;
+    m.maxP = std::max(m.maxP, L.proj.N); m.maxA = std::max(m.maxA, inner); m.maxCV = std::max(m.maxCV, C);
+    m.maxBG = std::max(m.maxBG, 2 * H);
+}
+
 struct MixerEntry;
 const MixerEntry & find_mixer(const std::string & type, size_t layer);
 void load_pair(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p);
@@ -588,6 +703,9 @@ const MixerEntry MIXERS[] = {
     { "parallel", MIX_PAIR, load_pair },
     { "chunk_attention", MIX_GQATTN, load_gqattn_chunks },
     { "window_attention", MIX_GQATTN, load_gqattn_window },
+    { "selective_scan", MIX_SELSCAN, load_selscan },
+    { "mlstm", MIX_MLSTM, load_mlstm },
+    { "mamba2", MIX_SSD, load_ssd },
 };
 
 const MixerEntry & find_mixer(const std::string & type, size_t layer) {
@@ -596,15 +714,14 @@ const MixerEntry & find_mixer(const std::string & type, size_t layer) {
 }
 
 // two mixers side by side on the same input: '<prefix>left.*' and '<prefix>right.*', each branch's output over its root mean
-// square times '<prefix>left.out' / '<prefix>right.out', then their mean. A branch names its mixer by "type" (absent: a sigmoid
-// attention on the left, a retention on the right).
+// square times '<prefix>left.out' / '<prefix>right.out', then their mean. A branch names its mixer by "type" (absent: the design's).
 void load_pair(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) {
-    const char * side[2] = { "left", "right" }, * dflt[2] = { "sigmoid_attention", "retention" };
+    const char * side[2] = { "left", "right" };
     L.parts.resize(2);
     L.n_rec = 0; L.cache_row = 0;
     for (int i = 0; i < 2; i++) {
         const Json & bj = mx.at(side[i]);
-        const MixerEntry & me = find_mixer(bj.string("type", dflt[i]), 0);
+        const MixerEntry & me = find_mixer(bj.string("type", m.pair_default[i]), 0);
         if (me.kind == MIX_PAIR) throw std::runtime_error("config: a branch of a parallel mixer cannot be a parallel mixer");
         LayerSpec & B = L.parts[(size_t) i];
         B.kind = me.kind;
@@ -788,13 +905,17 @@ DMat load_glu_pair(StackModel & m, const safetensors_file & sf, const std::strin
     if (into) { append(*into, W); return DMat(); }
     return up_mat(m, W, 2 * ff, E, nullptr);
 }
-// what a design fixes about its routed mixture: the score function, where a choice's weight is applied, a gate on the shared unit
-struct MixtureKind { int route_fn; bool scale_input; bool shared_gate; };
+// what a design fixes about its routed mixture: the score function, where a choice's weight is applied, a gate on the shared unit;
+// scores chosen with a correction and normalised, identity outputs, and clamped units (slope GLU_ALPHA, shift 1, "limit") instead of silu ones
+struct MixtureKind { int route_fn; bool scale_input; bool shared_gate; bool corrected = false; bool clamped = false; };
 void load_mixture(StackModel & m, LayerSpec & L, const Json & mj, const safetensors_file & sf, const std::string & p, const MixtureKind & mk) {
     const int E = m.E;
     L.route_fn = mk.route_fn; L.scale_input = mk.scale_input;
     const Json & rj = mj.at("router");
-    const int n = L.n_exp = need_int(rj, "experts"), top = L.top = need_int(rj, "top");
+    const int n_mat = L.n_exp = need_int(rj, "experts"), top = L.top = need_int(rj, "top");
+    L.n_ident = mk.corrected ? (int) rj.integer("identity", 0) : 0;
+    if (L.n_ident < 0) throw std::runtime_error("config: router.identity must not be negative");
+    const int n = n_mat + L.n_ident;                          // router outputs
     L.r_scale = (float) rj.number("scale", 1.0);
     L.n_groups = rj.has("groups") ? need_int(rj.at("groups"), "count") : 1;
     L.keep_groups = rj.has("groups") ? need_int(rj.at("groups"), "keep") : 1;
@@ -805,19 +926,24 @@ void load_mixture(StackModel & m, LayerSpec & L, const Json & mj, const safetens
     const int ff = L.e_ff = need_int(mj.at("expert"), "ff");
     L.ff_kind = FF_MOE;
     L.router = up_f32(m, sf.read_f32(p + "router", {n, E}));
+    if (mk.corrected) { L.corr = up_f32(m, sf.read_f32(p + "correction", {n})); L.norm_w = true; }
+    if (mk.clamped) L.e_limit = (float) mj.at("expert").number("limit");
+    else { L.act_alpha = 1.f; L.act_shift = 0.f; }
+    L.limit = INFINITY;
     std::vector<float> GU, DN;
-    for (int e = 0; e < n; e++) {
+    for (int e = 0; e < n_mat; e++) {
         const std::string ep = p + "e" + std::to_string(e) + ".";
         load_glu_pair(m, sf, ep, ff, E, &GU);
         append(DN, sf.read_f32(ep + "down", {E, ff}));
     }
     const int64_t before = m.weight_bytes;
-    L.e_gateup = up_mat(m, GU, 2 * ff, E, nullptr, n);
-    L.e_down = up_mat(m, DN, E, ff, nullptr, n);
-    m.weight_bytes = before + (m.weight_bytes - before) / n * top + (int64_t) n * E * 4;      // a token reads its chosen experts and the router
+    L.e_gateup = up_mat(m, GU, 2 * ff, E, nullptr, n_mat);
+    L.e_down = up_mat(m, DN, E, ff, nullptr, n_mat);
+    m.weight_bytes = before + (m.weight_bytes - before) / n_mat * std::min(top, n_mat) + (int64_t) n * E * 4;      // a token reads its chosen experts and the router
     L.ff = 0;
     if (mj.has("shared")) {
         const int sff = L.ff = need_int(mj.at("shared"), "ff");
+        if (mk.clamped) L.limit = (float) mj.at("shared").number("limit");
         L.gateup = load_glu_pair(m, sf, p + "shared.", sff, E, nullptr);
         L.down = up_mat(m, sf.read_f32(p + "shared.down", {E, sff}), E, sff, nullptr);
         if (mk.shared_gate) L.w_sg = up_f32(m, sf.read_f32(p + "shared.sg", {1, E}));
@@ -936,12 +1062,68 @@ void build_rumurax(StackModel & m, const Json & cfg, const safetensors_file & sf
     m.head = up_mat(m, sf.read_f32("head", {m.vocab, E}), m.vocab, E, nullptr);
 }
 
+// Kogerax: x = scale * embed -> layers (x += mult * norm1(mixer(x)); x += mult * norm2(ff(x)) when the layer has one; zero-centred norm
+// weights, the sub-layers read x itself) -> norm -> head
+void build_kogerax(StackModel & m, const Json & cfg, const safetensors_file & sf) {
+    m.block = BLOCK_POSTNORM;
+    m.unit_qk = true;
+    m.pair_default[0] = "window_attention"; m.pair_default[1] = "selective_scan";
+    m.vocab = need_int(cfg, "vocab"); m.E = need_int(cfg, "width");
+    m.eps = (float) cfg.at("norm").number("eps");
+    m.groups = 1;
+    m.residual_mult = (float) cfg.number("residual_mult", 1.0);
+    m.embed_scale = cfg.has("embedding") ? (float) cfg.at("embedding").number("scale", 1.0) : 1.f;
+    const int E = m.E;
+    const auto one_plus = [](std::vector<float> w) { for (float & v : w) v = 1.0f + v; return w; };
+    {
+        DMat d = up_mat(m, sf.read_f32("embed", {m.vocab, E}), m.vocab, E, nullptr);
+        m.embed = d.w;
+        m.weight_bytes -= d.bytes;
+    }
+    const Json & layers = cfg.at("layers");
+    if (layers.kind != Json::Arr || layers.arr.empty()) throw std::runtime_error("config: 'layers' must be a non-empty list");
+    const int n = (int) layers.arr.size();
+    for (int i = 0; i < n; i++) {
+        const Json & lj = layers.arr[(size_t) i];
+        const std::string type = lj.string("type", ""), p = "l" + std::to_string(i) + ".";
+        const MixerEntry * me = &find_mixer(type, (size_t) i);
+        if (me->kind != MIX_PAIR && me->kind != MIX_MLSTM && me->kind != MIX_SSD) throw std::runtime_error("config: mixer '" + type + "' is not part of the Kogerax design");
+        const int64_t bytes0 = m.weight_bytes;
+        m.layers.emplace_back();
+        LayerSpec & L = m.layers.back();
+        L.kind = me->kind;
+        L.has_mlp = lj.has("mlp");
+        L.norm1 = up_f32(m, one_plus(sf.read_f32(p + "norm1", {E})));
+        me->load(m, L, lj.at("mixer"), sf, p + "mix.");
+        if (L.has_mlp) {
+            const Json & mj = lj.at("mlp");
+            const std::string kind = mj.string("kind", "dense");
+            L.norm2 = up_f32(m, one_plus(sf.read_f32(p + "norm2", {E})));
+            if (kind == "moe") load_mixture(m, L, mj, sf, p + "mlp.", MixtureKind{0, false, true, true, true});
+            else if (kind == "dense") {
+                L.ff = need_int(mj, "ff");
+                L.act_kind = GLU_GELU;
+                L.gateup = load_glu_pair(m, sf, p + "mlp.", L.ff, E, nullptr);
+                L.down = up_mat(m, sf.read_f32(p + "mlp.down", {E, L.ff}), E, L.ff, nullptr);
+                m.maxA = std::max(m.maxA, L.ff);
+            } else throw std::runtime_error("config: feed-forward kind '" + kind + "' is not part of the Kogerax design (dense | moe)");
+        }
+        m.weight_bytes += (int64_t) E * 4 * ((L.has_mlp ? 2 : 1) + (L.kind == MIX_PAIR ? 2 : 0));
+        L.bytes = m.weight_bytes - bytes0;
+        m.weight_bytes = bytes0;
+        add_run(m, i, -1);
+    }
+    m.final_norm = up_f32(m, one_plus(sf.read_f32("final.norm", {E})));
+    m.head = up_mat(m, sf.read_f32("head", {m.vocab, E}), m.vocab, E, nullptr);
+}
+
 struct DesignEntry { const char * name; void (*build)(StackModel &, const Json &, const safetensors_file &); };
 const DesignEntry DESIGNS[] = {
     { "Matulorn", build_matulorn },
     { "Dopilorn", build_dopilorn },
     { "Tosevik", build_tosevik },
     { "Rumurax", build_rumurax },
+    { "Kogerax", build_kogerax },
 };
 
 // ---- launches ---------------------------------------------------------------------------------------------------------
@@ -958,12 +1140,14 @@ bool umma_enabled() {
 // bounded waits raise
 struct UmmaScratch { __nv_bfloat16 * xb = nullptr; size_t elems = 0; int * err = nullptr; };
 
-// what a product may ask for beyond its operands: the gated unit's constants (y = g sigmoid(alpha g) (u + shift), g and u clamped
-// at +-limit), rows sorted into segments per batch entry (tile kernels), an indexed batch (mat-vec)
+// what a product may ask for beyond its operands: the gated unit's kind and constants (y = g sigmoid(alpha g) (u + shift), g and u clamped
+// at +-limit, or gelu(g) u), rows sorted into segments per batch entry (tile kernels), an indexed batch (mat-vec)
 struct LinOpt {
     float alpha = GLU_ALPHA, shift = 1.f;
     const int32_t * seg = nullptr;
+    int glu_kind = GLU_SIGMOID;
     const int32_t * w_index = nullptr;
+    int n_w = 0;                            // mat-vec: matrices in the indexed batch (0: every index is one)
     int x_share = 1;
     const float * x_scale = nullptr;        // mat-vec: entry z runs on x_scale[z] times its input row
 };
@@ -971,8 +1155,8 @@ void linear_on(cudaStream_t st, int dtype, int64_t * launches, const float * X, 
                int T, int N, int K, int batch = 1, long long sX = 0, long long sW = 0, long long sY = 0, bool glu = false, float glu_limit = 0.f,
                const UmmaScratch * us = nullptr, const LinOpt * opt = nullptr) {
     if (T <= 0 || N <= 0) return;
-    LinArgs a{X, W, bias, Y, T, N, K, ldx, ldy, sX, sW, sY, 0, glu ? 1 : 0, glu_limit, GLU_ALPHA, 0, 0};
-    if (opt) { a.alpha = opt->alpha; a.up_shift = opt->shift; a.seg = opt->seg; a.w_index = opt->w_index; a.x_share = opt->x_share; a.x_scale = opt->x_scale; }
+    LinArgs a{X, W, bias, Y, T, N, K, ldx, ldy, sX, sW, sY, 0, glu ? GLU_SIGMOID : GLU_NONE, glu_limit, GLU_ALPHA, 0, 0};
+    if (opt) { if (glu) a.glu = opt->glu_kind; a.n_w = opt->n_w; a.alpha = opt->alpha; a.up_shift = opt->shift; a.seg = opt->seg; a.w_index = opt->w_index; a.x_share = opt->x_share; a.x_scale = opt->x_scale; }
     const int xbatch = a.seg ? 1 : batch;      // segments: X is one matrix of T rows
     const int vecw = dtype == STACK_F32 ? 4 : 8;
     const auto al16 = [](const void * p) { return ((uintptr_t) p & 15) == 0; };
@@ -1270,21 +1454,53 @@ void mixer_diffattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T)
     linear(c, c->A, H * V, L.o, c->out, E, T);
 }
 
-constexpr int RET_CHUNK_MIN_T = 128;      // shorter portions walk token by token
-size_t retention_chunk_smem(int D) { return ((size_t) 2 * RC * (D + 4) + (size_t) RC * (RC + 4) + (size_t) RC * 128 + RC + 1) * 4; }
-bool retention_chunks_enabled() {
+constexpr int SCAN_CHUNK_MIN_T = 128;     // shorter portions walk token by token
+size_t outer_chunk_smem(int D, int NC) { return ((size_t) 2 * RC * (D + 4) + (size_t) RC * (RC + 4) + (size_t) RC * NC) * 4; }
+bool scan_chunks_enabled() {
     static const bool on = [] { const char * e = std::getenv("BOOSTER_B200_STACK_RET_CHUNKS"); return !(e && e[0] == '0'); }();
     return on;
 }
 
 template <int DMAX>
-void launch_retention_scan(StackCtx * c, const LayerSpec & L, int T, int ldp, float * S) {
+void launch_outer_walk(StackCtx * c, const OuterScan & s) {
     // four lanes per column of the state; a head's columns are spread over blocks of >= 16 until the grid fills the SMs
-    int ncols = std::min(128, (L.V + 7) / 8 * 8);
-    while (ncols > 16 && L.H * ((L.V + ncols - 1) / ncols) < c->sm_count) ncols = (ncols / 2 + 7) / 8 * 8;
-    const int HD = L.H * L.D;
-    const dim3 grid((unsigned) L.H, (unsigned) ((L.V + ncols - 1) / ncols));
-    k_retention_scan<DMAX><<<grid, GD_RG * ncols, 0, c->st>>>(c->P, ldp, 0, HD, 2 * HD, L.decay, T, L.H, L.D, L.V, S, c->O);
+    const int cols = s.V + (s.norm ? 1 : 0);
+    int ncols = std::min(128, (cols + 7) / 8 * 8);
+    while (ncols > 16 && s.H * ((cols + ncols - 1) / ncols) < c->sm_count) ncols = (ncols / 2 + 7) / 8 * 8;
+    k_outer_scan<DMAX><<<dim3((unsigned) s.H, (unsigned) ((cols + ncols - 1) / ncols)), GD_RG * ncols, 0, c->st>>>(s);
+    c->launches++;
+}
+template <int NC>
+void launch_outer_chunks(StackCtx * c, const OuterScan & s) {
+    // per-chunk products in parallel, a short walk over the chunks in between
+    const int nch = (s.T + RC - 1) / RC, n = s.D * s.V + (s.norm ? s.D : 0);
+    const dim3 grid((unsigned) s.H, (unsigned) nch, (unsigned) ((s.V + NC - 1) / NC));
+    const auto al16 = [](const void * p) { return ((uintptr_t) p & 15) == 0; };
+    const int vec = ((s.ldq | s.ldk | s.ldv | s.D | s.V) & 3) == 0 && al16(s.Q) && al16(s.K) && al16(s.Vv) ? 1 : 0;
+    k_outer_chunk_kv<NC><<<grid, 256, 0, c->st>>>(s, vec, c->scan_sb, c->scan_ac);
+    k_outer_chunk_state<<<dim3((unsigned) s.H, (unsigned) ((n + 255) / 256)), 256, 0, c->st>>>(n, s.head_stride, nch, c->scan_ac, s.S, c->scan_sb);
+    k_outer_chunk_out<NC><<<grid, 128, outer_chunk_smem(s.D, NC), c->st>>>(s, vec, c->scan_sb);
+    c->launches += 3;
+}
+// the outer-product recurrence over a portion: long ones chunk by chunk, short ones token by token
+void outer_scan(StackCtx * c, const OuterScan & s) {
+    if (s.T >= SCAN_CHUNK_MIN_T && c->scan_sb && scan_chunks_enabled()) {
+        if (s.V <= 64) launch_outer_chunks<64>(c, s); else launch_outer_chunks<128>(c, s);
+    }
+    else if (s.D <= 32) launch_outer_walk<32>(c, s);
+    else if (s.D <= 64) launch_outer_walk<64>(c, s);
+    else if (s.D <= 128) launch_outer_walk<128>(c, s);
+    else launch_outer_walk<256>(c, s);
+}
+template <int KIND>
+void launch_outer_token(StackCtx * c, const OuterToken & t) {
+    const int threads = GD_RG * std::min(128, (t.V + 7) / 8 * 8);
+    const size_t sm = (size_t) (t.V + 1) * 4;
+    if (t.D <= 32) k_outer_token<32, KIND><<<t.H, threads, sm, c->st>>>(t);
+    else if (t.D <= 64) k_outer_token<64, KIND><<<t.H, threads, sm, c->st>>>(t);
+    else if (t.D <= 128) k_outer_token<128, KIND><<<t.H, threads, sm, c->st>>>(t);
+    else k_outer_token<256, KIND><<<t.H, threads, sm, c->st>>>(t);
+    c->launches++;
 }
 
 // retention: P[t] = [ q | k | v | gate ] -> rotation, key scale -> recurrence -> per-head unit norm, silu gate -> output product
@@ -1294,36 +1510,97 @@ void mixer_retention(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T
     linear(c, c->in, E, L.proj, c->P, ldp, T);
     if (T == 1) {
         // one token: rotation, state update, read-out norm and gate in one launch, a block per head
-        const RopeArgs rope{L.rope_freq, L.rope_dims, 1.0f};
-        const int threads = GD_RG * std::min(128, (V + 7) / 8 * 8);
-        const size_t sm = (size_t) V * 4;
-        const StepState * st = &c->d_step->st;
-        if (D <= 32) k_retention_token<32><<<H, threads, sm, c->st>>>(c->P, 0, HD, 2 * HD, 2 * HD + HV, L.decay, rope, L.k_scale, st, H, D, V, c->m->eps, S, c->A);
-        else if (D <= 64) k_retention_token<64><<<H, threads, sm, c->st>>>(c->P, 0, HD, 2 * HD, 2 * HD + HV, L.decay, rope, L.k_scale, st, H, D, V, c->m->eps, S, c->A);
-        else if (D <= 128) k_retention_token<128><<<H, threads, sm, c->st>>>(c->P, 0, HD, 2 * HD, 2 * HD + HV, L.decay, rope, L.k_scale, st, H, D, V, c->m->eps, S, c->A);
-        else k_retention_token<256><<<H, threads, sm, c->st>>>(c->P, 0, HD, 2 * HD, 2 * HD + HV, L.decay, rope, L.k_scale, st, H, D, V, c->m->eps, S, c->A);
-        c->launches++;
+        OuterToken t{};
+        t.P = c->P; t.q_off = 0; t.k_off = HD; t.v_off = 2 * HD; t.g_off = 2 * HD + HV;
+        t.decay = L.decay; t.rope = RopeArgs{L.rope_freq, L.rope_dims, 1.0f}; t.k_scale = L.k_scale; t.st = &c->d_step->st;
+        t.H = H; t.D = D; t.V = V; t.eps = c->m->eps; t.S = S; t.head_stride = (long long) L.head_stride; t.A = c->A;
+        launch_outer_token<TOKEN_RETENTION>(c, t);
         linear(c, c->A, HV, L.o, c->out, E, T);
         return;
     }
     k_retention_prep<<<dim3((unsigned) T, (unsigned) ((2 * H + 3) / 4)), 128, 0, c->st>>>(c->P, ldp, 0, HD, H, D, RopeArgs{L.rope_freq, L.rope_dims, 1.0f}, L.k_scale, &c->d_step->st);
-    if (T >= RET_CHUNK_MIN_T && c->ret_sb && retention_chunks_enabled()) {
-        // long portions: per-chunk products in parallel, a short walk over the chunks in between
-        const int nch = (T + RC - 1) / RC, vt = (V + 127) / 128;
-        const dim3 grid((unsigned) H, (unsigned) nch, (unsigned) vt);
-        const size_t sm = retention_chunk_smem(D);
-        k_retention_chunk_kv<<<grid, 256, 0, c->st>>>(c->P, ldp, HD, 2 * HD, L.decay, T, H, D, V, c->ret_sb);
-        k_retention_chunk_state<<<dim3((unsigned) H, (unsigned) ((D * V + 255) / 256)), 256, 0, c->st>>>(L.decay, T, D, V, nch, S, c->ret_sb);
-        k_retention_chunk_out<<<grid, 128, sm, c->st>>>(c->P, ldp, 0, HD, 2 * HD, L.decay, T, H, D, V, c->ret_sb, c->O);
-        c->launches += 2;
-    }
-    else if (D <= 32) launch_retention_scan<32>(c, L, T, ldp, S);
-    else if (D <= 64) launch_retention_scan<64>(c, L, T, ldp, S);
-    else if (D <= 128) launch_retention_scan<128>(c, L, T, ldp, S);
-    else launch_retention_scan<256>(c, L, T, ldp, S);
+    OuterScan s{};
+    s.Q = c->P; s.K = c->P + HD; s.Vv = c->P + 2 * HD; s.ldq = s.ldk = s.ldv = ldp;
+    s.T = T; s.H = H; s.share = 1; s.D = D; s.V = V; s.kind = SCAN_CONST; s.decay = L.decay; s.S = S; s.head_stride = (long long) L.head_stride; s.O = c->O;
+    outer_scan(c, s);
     k_delta_out<<<dim3((unsigned) T, (unsigned) ((H + 3) / 4)), 128, 0, c->st>>>(c->O, c->P, ldp, 2 * HD + HV, H, V, nullptr, 0, 0, c->m->eps, c->A);
-    c->launches += 3;
+    c->launches += 2;
     linear(c, c->A, HV, L.o, c->out, E, T);
+}
+
+// mLSTM: P[t] = [ q | k | v | output gate | input gate | forget gate ] -> gates, running maximum -> recurrence with a normaliser ->
+// per-head unit norm, weight, sigmoid gate -> output product
+void mixer_mlstm(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
+    const int E = c->m->E, H = L.H, D = L.D, V = L.V, HD = H * D, HV = H * V, ldp = L.proj.N, gi = 2 * HD + 2 * HV, ldg = 3 * H;
+    float * S = c->rec + R.off_rec, * m_state = S + (size_t) H * L.head_stride;
+    const float q_scale = (float) (1.0 / std::sqrt((double) D));
+    linear(c, c->in, E, L.proj, c->P, ldp, T);
+    if (T == 1) {
+        OuterToken t{};
+        t.P = c->P; t.q_off = 0; t.k_off = HD; t.v_off = 2 * HD; t.g_off = 2 * HD + HV; t.i_off = gi; t.f_off = gi + H;
+        t.q_scale = q_scale; t.cap = L.gate_cap; t.w = L.dnorm; t.m_state = m_state; t.m_stride = 1;
+        t.H = H; t.D = D; t.V = V; t.eps = c->m->eps; t.S = S; t.head_stride = (long long) L.head_stride; t.A = c->A;
+        launch_outer_token<TOKEN_MLSTM>(c, t);
+        linear(c, c->A, HV, L.o, c->out, E, T);
+        return;
+    }
+    k_mlstm_gates<<<H, 32, 0, c->st>>>(c->P, ldp, gi, gi + H, L.gate_cap, T, H, m_state, 1, c->BG, ldg);
+    OuterScan s{};
+    s.Q = c->P; s.K = c->P + HD; s.Vv = c->P + 2 * HD; s.ldq = s.ldk = s.ldv = ldp;
+    s.T = T; s.H = H; s.share = 1; s.D = D; s.V = V; s.kind = SCAN_TABLE; s.ab = c->BG; s.ld_ab = ldg; s.S = S; s.head_stride = (long long) L.head_stride;
+    s.norm = 1; s.O = c->O; s.den = c->den;
+    outer_scan(c, s);
+    k_mlstm_out<<<dim3((unsigned) T, (unsigned) ((H + 3) / 4)), 128, 0, c->st>>>(c->O, c->den, c->BG, ldg, q_scale, c->P, ldp, 2 * HD + HV, H, V, L.dnorm, c->m->eps, c->A);
+    c->launches += 2;
+    linear(c, c->A, HV, L.o, c->out, E, T);
+}
+
+// state-space duality: P[t] = [ z | x | B | C | dt ] -> convolution of x, B, C -> recurrence (keys B and queries C shared by a group's
+// heads, values x) -> skip, gate, norm in parts -> output product
+void mixer_ssd(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
+    const int E = c->m->E, H = L.H, N = L.D, V = L.V, G = L.KH, inner = L.inner, C = inner + 2 * G * N, ldp = L.proj.N;
+    float * S = c->rec + R.off_rec, * hist = S + ((size_t) H * N * V + 3) / 4 * 4;
+    linear(c, c->in, E, L.proj, c->P, ldp, T);
+    causal_conv(c, ConvArgs{c->P + inner, ldp, 0, L.wconv, 0, hist, 0, c->CV, C, 0, T, C, L.taps, 1, 0, nullptr, nullptr, 0, 0, 0, L.bconv});
+    OuterScan s{};
+    s.Vv = c->CV; s.K = c->CV + inner; s.Q = c->CV + inner + G * N; s.ldq = s.ldk = s.ldv = C;
+    s.T = T; s.H = H; s.share = H / G; s.D = N; s.V = V; s.S = S; s.head_stride = (long long) L.head_stride; s.O = c->O;
+    if (T == 1) { s.kind = SCAN_STEP; s.ab = c->P + inner + C; s.ld_ab = ldp; s.dt_bias = L.dt_bias; s.A_log = L.A_log; }
+    else {
+        k_step_table<<<T, H >= 128 ? 128 : 32, 0, c->st>>>(c->P + inner + C, ldp, L.dt_bias, L.A_log, H, c->BG, 2 * H);
+        c->launches++;
+        s.kind = SCAN_TABLE; s.ab = c->BG; s.ld_ab = 2 * H;
+    }
+    outer_scan(c, s);
+    const int n = inner / L.norm_parts, nt = T > 16 ? 256 : std::min(1024, std::max(128, (n + 63) / 64 * 32));
+    k_gated_part_norm<<<dim3((unsigned) T, (unsigned) L.norm_parts), nt, 0, c->st>>>(c->O, c->CV, C, L.skip, c->P, ldp, inner, V, L.norm_parts, L.dnorm, c->m->eps, c->A);
+    c->launches++;
+    linear(c, c->A, inner, L.o, c->out, E, T);
+}
+
+template <int LANES, int NS>
+void launch_selective(StackCtx * c, const LayerSpec & L, const SelScan & s) {
+    const int nblk = (s.inner + 256 / LANES - 1) / (256 / LANES);
+    if (s.T > 1) k_selective_scan<LANES, NS><<<nblk, 256, 0, c->st>>>(s);
+    else if (c->m->dtype == STACK_F32) k_selective_token<float, LANES, NS><<<nblk, 256, (size_t) L.dt_rank * 4, c->st>>>(s, (const float *) L.wdt.w, L.wdt.bias, L.dt_rank);
+    else k_selective_token<__nv_bfloat16, LANES, NS><<<nblk, 256, (size_t) L.dt_rank * 4, c->st>>>(s, (const __nv_bfloat16 *) L.wdt.w, L.wdt.bias, L.dt_rank);
+    c->launches++;
+}
+// selective scan: P[t] = [ x | z ] -> convolution of x -> [ step latent | B | C ] from it -> step sizes -> scan with skip and gate -> output product
+void mixer_selscan(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
+    const int E = c->m->E, n = L.inner, N = L.state, ldb = (L.dt_rank + 2 * N + 3) / 4 * 4;
+    float * S = c->rec + R.off_rec, * hist = S + (size_t) n * N;
+    linear(c, c->in, E, L.proj, c->P, 2 * n, T);
+    causal_conv(c, ConvArgs{c->P, 2 * n, 0, L.wconv, 0, hist, 0, c->CV, n, 0, T, n, L.taps, 1, 0, nullptr, nullptr, 0, 0, 0, L.bconv});
+    linear(c, c->CV, n, L.wx, c->BG, ldb, T);
+    if (T > 1) linear(c, c->BG, ldb, L.wdt, c->O, n, T);
+    const SelScan s{c->CV, n, c->O, n, c->BG, ldb, L.dt_rank, L.dt_rank + N, c->P + n, 2 * n, L.A_log, L.skip, S, T, n, N, c->A};
+    if (N <= 16) launch_selective<4, 4>(c, L, s);
+    else if (N <= 32) launch_selective<8, 4>(c, L, s);
+    else if (N <= 64) launch_selective<16, 4>(c, L, s);
+    else if (N <= 128) launch_selective<16, 8>(c, L, s);
+    else launch_selective<32, 8>(c, L, s);
+    linear(c, c->A, n, L.o, c->out, E, T);
 }
 
 constexpr int SIG_MAX_SPLIT = 16;
@@ -1393,7 +1670,7 @@ void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
     const StepState * st = &c->d_step->st;
     linear(c, c->in, E, L.proj, c->P, ldp, T);
     const GqaPrepArgs pa{c->P, ldp, H, G, D, V, L.qw, L.kw, c->m->eps, RopeArgs{L.rope_freq, L.rope_dims, 1.0f, L.rope_adjacent ? 1 : 0}, st, c->CV, cache, row,
-                         c->VF, L.vmode, L.vlambda};
+                         c->VF, L.vmode, L.vlambda, L.unit_qk ? 1 : 0};
     k_gqa_prep<<<dim3((unsigned) T, T <= 16 ? (unsigned) ((H + G + 7) / 8) : 1u), 256, 0, c->st>>>(pa);      // few tokens: a token's heads over several blocks
     c->launches++;
     if (L.pool > 0) { k_pool_rows<<<dim3((unsigned) (T / L.pool + 1), (unsigned) ((row + 127) / 128)), 128, 0, c->st>>>(cache, row, pool, L.pool, st); c->launches++; }
@@ -1479,6 +1756,9 @@ void run_mixer(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
         case MIX_SIGATTN:   mixer_sigattn(c, L, R, T); break;
         case MIX_PAIR:      mixer_pair(c, L, R, T); break;
         case MIX_GQATTN:    mixer_gqattn(c, L, R, T); break;
+        case MIX_SELSCAN:   mixer_selscan(c, L, R, T); break;
+        case MIX_MLSTM:     mixer_mlstm(c, L, R, T); break;
+        case MIX_SSD:       mixer_ssd(c, L, R, T); break;
         case MIX_MINGRU:   mixer_mingru(c, L, R, T); break;
         case MIX_LATENT:   mixer_latent(c, L, R, T); break;
         case MIX_DELTA:    mixer_delta(c, L, R, T); break;
@@ -1573,42 +1853,43 @@ void enqueue_layers_parallel(StackCtx * c, int T) {
     SCU(cudaGetLastError());
 }
 
-// routed mixture on c->Hn (a design whose experts run on the weighted input gets outputs that are added as they are): the chosen experts' outputs by slot in c->Yk (slot order in *slot_of: nullptr = t top + k), the
-// shared unit's in c->Y; the layer's join weighs and adds them
-void mixture_ff(StackCtx * c, const LayerSpec & L, int T, const int32_t ** slot_of) {
-    const int E = c->m->E, top = L.top, ff = L.e_ff, slots = T * top;
-    const RouteArgs ra{c->Hn, E, E, L.router, L.w_sg, L.n_exp, top, L.n_groups, L.keep_groups, L.r_scale, c->r_sel, c->r_wt, c->r_sg, c->r_z, c->r_counter, L.route_fn, T <= 16 ? 8 : 1};
-    k_moe_route<<<dim3((unsigned) T, (unsigned) ((L.n_exp + (L.w_sg ? 1 : 0) + 8 / ra.wpr - 1) / (8 / ra.wpr))), 256, (size_t) (2 * L.n_exp + L.n_groups) * 4, c->st>>>(ra);
+// routed mixture on the rows h (a design whose experts run on the weighted input gets outputs that are added as they are): the chosen
+// experts' outputs by slot in c->Yk (slot order in *slot_of: nullptr = t top + k; slots of identity outputs are left alone), the shared
+// unit's in c->Y; the layer's join weighs and adds them
+void mixture_ff(StackCtx * c, const LayerSpec & L, const float * h, int T, const int32_t ** slot_of) {
+    const int E = c->m->E, top = L.top, ff = L.e_ff, slots = T * top, n = L.n_exp + L.n_ident;
+    const RouteArgs ra{h, E, E, L.router, L.w_sg, n, top, L.n_groups, L.keep_groups, L.r_scale, c->r_sel, c->r_wt, c->r_sg, c->r_z, c->r_counter, L.route_fn, T <= 16 ? 8 : 1, L.corr, L.norm_w ? 1 : 0};
+    k_moe_route<<<dim3((unsigned) T, (unsigned) ((n + (L.w_sg ? 1 : 0) + 8 / ra.wpr - 1) / (8 / ra.wpr))), 256, (size_t) (2 * n + L.n_groups) * 4, c->st>>>(ra);
     c->launches++;
     LinOpt o;
-    o.alpha = 1.f; o.shift = 0.f;               // silu(gate) * up, no clamp
+    o.glu_kind = L.act_kind; o.alpha = L.act_alpha; o.shift = L.act_shift;
     if (T <= GEMV_MAX_T) {
         // few tokens: one mat-vec per (token, choice) against the chosen expert's matrices
-        o.w_index = c->r_sel; o.x_share = top;
+        o.w_index = c->r_sel; o.n_w = L.n_exp; o.x_share = top;
         if (L.scale_input) o.x_scale = c->r_wt;     // W (w h) = w (W h): the weight meets the products before the gated unit
-        linear(c, c->Hn, E, L.e_gateup, c->Ap, ff, 1, slots, E, ff, true, INFINITY, &o);
+        linear(c, h, E, L.e_gateup, c->Ap, ff, 1, slots, E, ff, true, L.e_limit, &o);
         o.x_share = 1; o.x_scale = nullptr;
         linear(c, c->Ap, ff, L.e_down, c->Yk, E, 1, slots, ff, E, false, 0.f, &o);
         *slot_of = nullptr;
     } else {
         // prompt portion: rows sorted by expert, one segmented product per projection
         int tpe = 1;
-        while (tpe * 2 * L.n_exp <= 1024 && tpe * 2 <= slots) tpe *= 2;
-        const size_t cnt_bytes = (size_t) L.n_exp * tpe * 4;
+        while (tpe * 2 * n <= 1024 && tpe * 2 <= slots) tpe *= 2;
+        const size_t cnt_bytes = (size_t) n * tpe * 4;
         const int in_smem = (size_t) slots * 4 + cnt_bytes <= 40 * 1024 ? 1 : 0;
-        k_moe_sort<<<1, 1024, cnt_bytes + (in_smem ? (size_t) slots * 4 : 0), c->st>>>(c->r_sel, slots, top, L.n_exp, tpe, in_smem, c->r_seg, c->r_slot, c->r_src);
-        if (L.scale_input) k_spread_rows<<<slots, 128, 0, c->st>>>(c->Hn, E, c->r_slot, c->r_wt, top, E, c->Xp);
-        else k_gather_rows<<<slots, 128, 0, c->st>>>(c->Hn, E, c->r_src, E, c->Xp);
+        k_moe_sort<<<1, 1024, cnt_bytes + (in_smem ? (size_t) slots * 4 : 0), c->st>>>(c->r_sel, slots, top, n, tpe, in_smem, c->r_seg, c->r_slot, c->r_src);
+        if (L.scale_input) k_spread_rows<<<slots, 128, 0, c->st>>>(h, E, c->r_slot, c->r_wt, top, E, c->Xp);
+        else k_gather_rows<<<slots, 128, 0, c->st>>>(h, E, c->r_src, E, c->Xp);
         c->launches += 2;
         o.seg = c->r_seg;
-        linear(c, c->Xp, E, L.e_gateup, c->Ap, ff, slots, L.n_exp, 0, 0, true, INFINITY, &o);
+        linear(c, c->Xp, E, L.e_gateup, c->Ap, ff, slots, L.n_exp, 0, 0, true, L.e_limit, &o);      // rows of identity outputs sort behind the last matrix
         linear(c, c->Ap, ff, L.e_down, c->Yk, E, slots, L.n_exp, 0, 0, false, 0.f, &o);
         *slot_of = c->r_slot;
     }
     if (L.ff > 0) {
         LinOpt s;
-        s.alpha = 1.f; s.shift = 0.f;
-        linear(c, c->Hn, E, L.gateup, c->A, L.ff, T, 1, 0, 0, true, INFINITY, &s);
+        s.glu_kind = L.act_kind; s.alpha = L.act_alpha; s.shift = L.act_shift;
+        linear(c, h, E, L.gateup, c->A, L.ff, T, 1, 0, 0, true, L.limit, &s);
         linear(c, c->A, L.ff, L.down, c->Y, E, T);
     }
 }
@@ -1646,7 +1927,7 @@ void enqueue_layers_prenorm(StackCtx * c, int T) {
         if (L.has_mlp) {
             JoinArgs f{};
             f.X = c->X; f.E = E; f.eps = m.eps;
-            mixture_ff(c, L, T, &f.slot_of);
+            mixture_ff(c, L, c->Hn, T, &f.slot_of);
             f.Yk = c->Yk; f.wt = c->r_wt; f.top = L.top;
             if (L.ff > 0) { f.Ysh = c->Y; f.sg = c->r_sg; }
             layer_end(f);
@@ -1694,10 +1975,55 @@ void enqueue_layers_hyper(StackCtx * c, int T) {
         join(0, j);
         if (L.has_mlp) {
             HcJoinArgs f{};
-            mixture_ff(c, L, T, &f.slot_of);
+            mixture_ff(c, L, c->Hn, T, &f.slot_of);
             f.Yk = c->Yk; f.top = L.top;
             if (L.ff > 0) f.Ya = c->Y;
             join(1, f);
+        }
+        if (c->taps) tap_layer(c, ri, T);
+    }
+    SCU(cudaGetLastError());
+}
+
+// blocks normed on the way out: x += mult * norm1(mixer(x)); x += mult * norm2(ff(x)), the sub-layers reading x itself. Every sub-layer
+// ends in one k_post_join launch; the last one also leaves the model's norm of x in c->Hn for the head.
+void enqueue_layers_postnorm(StackCtx * c, int T) {
+    StackModel & m = *c->m;
+    const int E = m.E;
+    if (m.dtype == STACK_F32) k_embed_plain<float><<<T, hc_threads(T, E), 0, c->st>>>((const float *) m.embed, c->d_step->tokens, E, m.vocab, c->X, nullptr, 0, m.embed_scale);
+    else k_embed_plain<__nv_bfloat16><<<T, hc_threads(T, E), 0, c->st>>>((const __nv_bfloat16 *) m.embed, c->d_step->tokens, E, m.vocab, c->X, nullptr, 0, m.embed_scale);
+    c->launches++;
+    for (size_t ri = 0; ri < m.runs.size(); ri++) {
+        const RunSpec & R = m.runs[ri];
+        const LayerSpec & L = m.layers[(size_t) R.layer];
+        const bool last = ri + 1 == m.runs.size();
+        const auto join = [&](PostJoinArgs & j, const float * w, bool end) {
+            j.X = c->X; j.E = E; j.eps = m.eps; j.mult = m.residual_mult; j.w = w; j.scratch = c->Hn;
+            if (end && last) { j.fw = m.final_norm; j.Hn = c->Hn; }
+            if (E % 4 == 0) k_post_join<4><<<T, hc_threads(T, E, 4), 0, c->st>>>(j);      // every buffer of a context is 16-byte aligned and its rows are E floats apart
+            else k_post_join<1><<<T, hc_threads(T, E), 0, c->st>>>(j);
+            c->launches++;
+        };
+        c->in = c->X; c->out = c->Y;
+        run_mixer(c, L, R, T);
+        PostJoinArgs j{};
+        j.Ya = c->Y;
+        if (L.kind == MIX_PAIR) { j.Yb = c->Y2; j.wa = L.pair_w[0]; j.wb = L.pair_w[1]; }
+        join(j, L.norm1, !L.has_mlp);
+        if (L.has_mlp) {
+            PostJoinArgs f{};
+            if (L.ff_kind == FF_MOE) {
+                mixture_ff(c, L, c->X, T, &f.slot_of);
+                f.Yk = c->Yk; f.wt = c->r_wt; f.sel = c->r_sel; f.top = L.top; f.n_real = L.n_exp;
+                if (L.ff > 0) { f.Ysh = c->Y; f.sg = c->r_sg; }
+            } else {
+                LinOpt o;
+                o.glu_kind = L.act_kind;
+                linear(c, c->X, E, L.gateup, c->A, L.ff, T, 1, 0, 0, true, INFINITY, &o);
+                linear(c, c->A, L.ff, L.down, c->Y, E, T);
+                f.Ya = c->Y;
+            }
+            join(f, L.norm2, true);
         }
         if (c->taps) tap_layer(c, ri, T);
     }
@@ -1709,14 +2035,15 @@ void enqueue_layers(StackCtx * c, int T) {
     if (c->m->block == BLOCK_PARALLEL) enqueue_layers_parallel(c, T);
     else if (c->m->block == BLOCK_PRENORM) enqueue_layers_prenorm(c, T);
     else if (c->m->block == BLOCK_HYPER) enqueue_layers_hyper(c, T);
+    else if (c->m->block == BLOCK_POSTNORM) enqueue_layers_postnorm(c, T);
     else enqueue_layers_sequential(c, T);
 }
 
 // final norm + head on n_rows rows of the pass (row indices in d_step->rows) -> d_logits[row_off ..]
 void enqueue_head(StackCtx * c, int n_rows, int64_t row_off, bool one_token = false) {
     StackModel & m = *c->m;
-    if (m.block == BLOCK_HYPER) {
-        // the last join left the normed sum of the streams in Hn for every row of the pass: the wanted rows are gathered for the head
+    if (m.block == BLOCK_HYPER || m.block == BLOCK_POSTNORM) {
+        // the last join left the normed residual (the sum of the streams) in Hn for every row of the pass: the wanted rows are gathered for the head
         const float * hn = c->Hn;
         if (!one_token) { k_gather_rows<<<n_rows, 128, 0, c->st>>>(c->Hn, m.E, c->d_step->rows, m.E, c->Y); c->launches++; hn = c->Y; }
         linear(c, hn, m.E, m.head, c->d_logits + row_off * m.vocab, m.vocab, n_rows);
@@ -1819,7 +2146,7 @@ void stack_ctx_free(StackCtx * c) {
     cudaFree(c->d_out_tokens); cudaFree(c->d_counter);
     for (float * p : c->pools) cudaFree(p);
     for (float * p : { c->XS, c->VF }) cudaFree(p);
-    for (float * p : { c->Y2, c->U, c->XC, c->keep, c->ret_sb, c->Xp, c->Ap, c->Yk, c->r_wt, c->r_sg, c->r_z }) cudaFree(p);
+    for (float * p : { c->Y2, c->U, c->XC, c->keep, c->scan_sb, c->scan_ac, c->den, c->Xp, c->Ap, c->Yk, c->r_wt, c->r_sg, c->r_z }) cudaFree(p);
     cudaFree(c->r_counter);
     for (int32_t * p : { c->r_sel, c->r_slot, c->r_src, c->r_seg }) cudaFree(p);
     for (float * p : { c->X, c->Hn, c->Y, c->P, c->A, c->QK, c->OL, c->CV, c->BG, c->O, c->rec, c->d_logits }) cudaFree(p);
@@ -1851,11 +2178,17 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
         if (m->depth_avg) fl(&c->keep, (m->layers.size() + 1) * cap * m->E);
         if (m->block == BLOCK_HYPER) fl(&c->XS, (size_t) m->streams * cap * m->E);
         if (m->vfirst_width > 0) fl(&c->VF, cap * (size_t) m->vfirst_width);
-        if (m->max_ret_state > 0 && c->cap >= RET_CHUNK_MIN_T) {
-            fl(&c->ret_sb, (size_t) ((c->cap + RC - 1) / RC) * m->max_ret_state);
+        if (m->max_scan_heads > 0) fl(&c->den, cap * (size_t) m->max_scan_heads);
+        if (m->max_scan_state > 0 && c->cap >= SCAN_CHUNK_MIN_T) {
+            const size_t nch = (size_t) (c->cap + RC - 1) / RC;
+            fl(&c->scan_sb, nch * m->max_scan_state); fl(&c->scan_ac, nch * (size_t) m->max_scan_heads);
             static size_t attr = 48 * 1024;
-            const size_t need = retention_chunk_smem(m->max_ret_dim);
-            if (need > attr) { SCU(cudaFuncSetAttribute(k_retention_chunk_out, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) need)); attr = need; }
+            const size_t need = outer_chunk_smem(m->max_scan_dim, 128);
+            if (need > attr) {
+                SCU(cudaFuncSetAttribute(k_outer_chunk_out<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) need));
+                SCU(cudaFuncSetAttribute(k_outer_chunk_out<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) need));
+                attr = need;
+            }
         }
         size_t moe_rows = 0;
         if (m->max_slots > 0) {

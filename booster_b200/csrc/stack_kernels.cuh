@@ -36,6 +36,16 @@ __device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
+// VEC = 4: rows are walked in 16-byte chunks (E a multiple of 4, 16-byte aligned rows); VEC = 1: any E.
+template <int VEC> __device__ __forceinline__ void ld_chunk(const float * p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) { const float4 f = *reinterpret_cast<const float4 *>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+    else v[0] = p[0];
+}
+template <int VEC> __device__ __forceinline__ void st_chunk(float * p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else p[0] = v[0];
+}
+
 // what a step works on: written by the host (or by a memcpy node of the replayed decode graph) before the launches
 struct StepState {
     int32_t pos0;       // position of the step's first token within its sequence
@@ -145,26 +155,33 @@ struct LinArgs {
     int T, N, K, ldx, ldy;
     long long sX, sW, sY;
     int vec;            // 1: K, ldx and all bases allow 16-byte loads
-    int glu;            // 1: rows of W are interleaved (2i: gate_i, 2i + 1: up_i); the epilogue writes the clamped gated unit
-    float limit, alpha; //    y_i = g sigmoid(alpha g) (u + 1), g = min(gate_i, limit), u = clamp(up_i, -limit, limit), to Y[t][i] (N / 2 wide)
+    int glu;            // GLU_*: rows of W are interleaved (2i: gate_i, 2i + 1: up_i); the epilogue writes a gated unit to Y[t][i] (N / 2 wide)
+    float limit, alpha; //    GLU_SIGMOID: y_i = g sigmoid(alpha g) (u + up_shift), g = min(gate_i, limit), u = clamp(up_i, -limit, limit); GLU_GELU: gelu(gate_i) up_i
     int w_kn, ldw;      // k_gemm_simt only. w_kn = 1: W is given [K][N] with row stride ldw (the attention's weights x cached rows);
                         // w_kn = 0 and ldw > 0: W is [N][K] with row stride ldw (keys inside wider cached rows)
     int nz2 = 1;        // k_gemm_simt only: blockIdx.z = z1 * nz2 + z2, a second batch level with the strides below
     long long sX2 = 0, sW2 = 0, sY2 = 0;
-    float up_shift = 1.0f;                  // the gated unit's (u + up_shift)
+    float up_shift = 1.0f;
     // tile kernels: batch entry z works on rows seg[z] .. seg[z + 1] - 1 of X and Y (rows sorted by the matrix they meet: a routed
     // mixture's experts); T is then only the most rows an entry can have
     const int32_t * seg = nullptr;
     // k_gemv: entry z meets matrix w_index[z] of the batch and reads the rows of entry z / x_share
     const int32_t * w_index = nullptr;
+    int n_w = 0;        // > 0: matrices in the batch; an entry that names another one is left alone (a routed choice without a matrix)
     int x_share = 1;
     // k_gemv: entry z's input row is x_scale[z] times the row it reads (a routed expert that runs on a weighted input); no bias then
     const float * x_scale = nullptr;
     int accum = 0;      // k_gemm_simt only: Y += the product (a second set of keys joining a weighted sum)
 };
+enum { GLU_NONE = 0, GLU_SIGMOID = 1, GLU_GELU = 2 };
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, float alpha, float shift) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);      // limit = +inf: no clamp
     return g * sigmoidf_(alpha * g) * (u + shift);
+}
+// gelu in its tanh form: z/2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float gelu_tanhf_(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
+__device__ __forceinline__ float gated_unit(const LinArgs & a, float gate, float up) {
+    return a.glu == GLU_GELU ? gelu_tanhf_(gate) * up : clamped_glu(gate, up, a.limit, a.alpha, a.up_shift);
 }
 
 constexpr int GEMV_MAX_T = 4;
@@ -174,7 +191,9 @@ __global__ void __launch_bounds__(256) k_gemv(const LinArgs a) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int n = (blockIdx.x * (blockDim.x >> 5) + warp) * RPW;      // RPW = 2: a (gate, up) pair per warp
     if (n >= a.N) return;
-    const WT * w = reinterpret_cast<const WT *>(a.W) + (size_t) (a.w_index ? a.w_index[blockIdx.z] : blockIdx.z) * a.sW + (size_t) n * a.K;
+    const int wi = a.w_index ? a.w_index[blockIdx.z] : (int) blockIdx.z;
+    if (a.n_w > 0 && wi >= a.n_w) return;
+    const WT * w = reinterpret_cast<const WT *>(a.W) + (size_t) wi * a.sW + (size_t) n * a.K;
     const float * x = a.X + (size_t) (blockIdx.z / a.x_share) * a.sX;
     float acc[RPW][GEMV_MAX_T];
 #pragma unroll
@@ -244,7 +263,7 @@ __global__ void __launch_bounds__(256) k_gemv(const LinArgs a) {
             for (int r = 0; r < RPW; r++) s[r] = warp_sum(acc[r][t]) * (a.x_scale ? a.x_scale[blockIdx.z] : 1.0f) + (a.bias ? a.bias[n + r] : 0.f);
             if (lane == 0) {
                 float * y = a.Y + (size_t) blockIdx.z * a.sY + (size_t) t * a.ldy;
-                if constexpr (RPW == 2) y[n >> 1] = clamped_glu(s[0], s[1], a.limit, a.alpha, a.up_shift);
+                if constexpr (RPW == 2) y[n >> 1] = gated_unit(a, s[0], s[1]);
                 else y[n] = s[0];
             }
         }
@@ -331,7 +350,7 @@ __global__ void __launch_bounds__(256) k_gemm_simt(const LinArgs a) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
-                if (n + 1 < a.N) Y[(size_t) m * a.ldy + (n >> 1)] = clamped_glu(acc[i][j] + (a.bias ? a.bias[n] : 0.f), acc[i][j + 1] + (a.bias ? a.bias[n + 1] : 0.f), a.limit, a.alpha, a.up_shift);
+                if (n + 1 < a.N) Y[(size_t) m * a.ldy + (n >> 1)] = gated_unit(a, acc[i][j] + (a.bias ? a.bias[n] : 0.f), acc[i][j + 1] + (a.bias ? a.bias[n + 1] : 0.f));
             }
             continue;
         }
@@ -522,7 +541,7 @@ __global__ void __launch_bounds__(256) k_gemm_bf16_mma(const LinArgs a) {
                 const int n = n0 + wn + 8 * j + (lane & 3) * 2 + (e & 1);
                 if (a.glu) {            // this thread holds the (gate, up) pair of unit n / 2 in elements e, e + 1
                     if (!(e & 1) && m < T && n + 1 < a.N)
-                        Y[(size_t) m * a.ldy + (n >> 1)] = clamped_glu(acc[i][j][e] + (a.bias ? a.bias[n] : 0.f), acc[i][j][e + 1] + (a.bias ? a.bias[n + 1] : 0.f), a.limit, a.alpha, a.up_shift);
+                        Y[(size_t) m * a.ldy + (n >> 1)] = gated_unit(a, acc[i][j][e] + (a.bias ? a.bias[n] : 0.f), acc[i][j][e + 1] + (a.bias ? a.bias[n + 1] : 0.f));
                 } else if (m < T && n < a.N) Y[(size_t) m * a.ldy + n] = acc[i][j][e] + (a.bias ? a.bias[n] : 0.f);
             }
 }
@@ -672,7 +691,7 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
                 for (int j = 0; j < 16; j += 2) {
                     const int n = n0 + cbase + c + j;
                     if (a.glu) {
-                        if (n + 1 < a.N) Y[n >> 1] = clamped_glu(v[j] + (a.bias ? a.bias[n] : 0.f), v[j + 1] + (a.bias ? a.bias[n + 1] : 0.f), a.limit, a.alpha, a.up_shift);
+                        if (n + 1 < a.N) Y[n >> 1] = gated_unit(a, v[j] + (a.bias ? a.bias[n] : 0.f), v[j + 1] + (a.bias ? a.bias[n + 1] : 0.f));
                     } else {
                         if (n < a.N) Y[n] = v[j] + (a.bias ? a.bias[n] : 0.f);
                         if (n + 1 < a.N) Y[n + 1] = v[j + 1] + (a.bias ? a.bias[n + 1] : 0.f);
@@ -1093,7 +1112,7 @@ __global__ void k_latent_softmax_rows(float * __restrict__ S, int n_rows, int H,
 
 // ---- causal convolution over time on each channel ----------------------------------------------------------------------------
 // y_t = sum_k w[c][k] x_(t - taps + 1 + k): the last weight is the current token's, inputs before the sequence's start are zero,
-// no bias. hist holds the taps - 1 inputs before the portion ([taps - 1][C]); it is part of the sequence's state and is moved
+// a bias per channel when given. hist holds the taps - 1 inputs before the portion ([taps - 1][C]); it is part of the sequence's state and is moved
 // on by k_causal_conv_hist after the portion. act: 0 none, 1 silu. add_input: Y = X + conv(X) (a convolution around a
 // residual path). blockIdx.z runs over a batch of independent convolutions (element strides sX / sW / sH / sY). Channels from
 // `split` on can be written to the row of the token's position in a per-position cache instead of Y (an attention's keys and
@@ -1106,6 +1125,7 @@ struct ConvArgs {
     int T, C, taps, act, add_input;
     const StepState * st; float * cache; int ldc, split;      // cache == nullptr: everything goes to Y
     int fuse_hist;                                            // T == 1: the thread also moves its channel's history on (no second launch)
+    const float * bias = nullptr;
 };
 __global__ void k_causal_conv(const ConvArgs a) {
     const int c = blockIdx.x * blockDim.x + threadIdx.x, t = blockIdx.y, z = blockIdx.z;
@@ -1113,7 +1133,7 @@ __global__ void k_causal_conv(const ConvArgs a) {
     const float * X = a.X + (size_t) z * a.sX;
     const float * w = a.w + (size_t) z * a.sW + (size_t) c * a.taps;
     const float * hist = a.hist + (size_t) z * a.sH;
-    float y = 0.f;
+    float y = a.bias ? a.bias[c] : 0.f;
     for (int k = 0; k < a.taps; k++) {
         const int tau = t - (a.taps - 1) + k;
         const float in = tau >= 0 ? X[(size_t) tau * a.ldx + c] : hist[(size_t) (a.taps - 1 + tau) * a.C + c];
@@ -1631,14 +1651,14 @@ k_add_norm2_canon1(float * __restrict__ X, const float * __restrict__ Ya, const 
     }
 }
 
-// embedding without a norm: X[t] = embed[token[t]]; X0 (row stride ld0), when given, keeps the same row for later layers
+// embedding without a norm: X[t] = scale * embed[token[t]]; X0 (row stride ld0), when given, keeps the same row for later layers
 template <typename WT>
-__global__ void k_embed_plain(const WT * __restrict__ embed, const int32_t * __restrict__ tokens, int E, int n_vocab, float * __restrict__ X, float * __restrict__ X0, int ld0) {
+__global__ void k_embed_plain(const WT * __restrict__ embed, const int32_t * __restrict__ tokens, int E, int n_vocab, float * __restrict__ X, float * __restrict__ X0, int ld0, float scale = 1.0f) {
     const int t = blockIdx.x;
     int tok = tokens[t];
     tok = tok < 0 ? 0 : tok >= n_vocab ? n_vocab - 1 : tok;
     for (int i = threadIdx.x; i < E; i += blockDim.x) {
-        const float v = wf(embed, (size_t) tok * E + i);
+        const float v = scale * wf(embed, (size_t) tok * E + i);
         X[(size_t) t * E + i] = v;
         if (X0) X0[(size_t) t * ld0 + i] = v;
     }

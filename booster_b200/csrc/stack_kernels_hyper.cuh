@@ -75,15 +75,6 @@ struct HcJoinArgs {
     float nin[HC_MAX]; float g; float eps; float * Hn;
     float * Xsum;
 };
-// VEC = 4: rows are walked in 16-byte chunks (E a multiple of 4, 16-byte aligned rows); VEC = 1: any E.
-template <int VEC> __device__ __forceinline__ void ld_chunk(const float * p, float (&v)[VEC]) {
-    if constexpr (VEC == 4) { const float4 f = *reinterpret_cast<const float4 *>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
-    else v[0] = p[0];
-}
-template <int VEC> __device__ __forceinline__ void st_chunk(float * p, const float (&v)[VEC]) {
-    if constexpr (VEC == 4) *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
-    else p[0] = v[0];
-}
 constexpr int HC_OWN = 2;              // read-in chunks a thread keeps in registers until the row's sum of squares is known
 template <int VEC>
 __global__ void __launch_bounds__(VEC == 4 ? 512 : 1024) k_hc_join(const HcJoinArgs a) {
@@ -157,7 +148,8 @@ __global__ void __launch_bounds__(VEC == 4 ? 512 : 1024) k_hc_join(const HcJoinA
 // ---- soft-max attention over grouped key/value heads ------------------------------------------------------------------------------
 // P[t] = [ q: H x D | k: G x D | v: G x V | ... ]. Query head h reads key/value head h / (H / G).
 // Step 1, per token: every q and k head over its own root mean square (eps inside the root) times a weight [D] shared by the heads
-// (qw / kw; nullptr: no norm), then the rotation of the first rope.dims entries by the token's position. Queries go to Q[t]
+// (qw / kw; nullptr: no norm, or with `unit` the norm without a weight — the rotation turns pairs and leaves the root mean square as it
+// is, so the order of the two does not matter), then the rotation of the first rope.dims entries by the token's position. Queries go to Q[t]
 // (H x D), keys and values to the cache row of the position: [ k: G x D | v: G x V ]. Values: vmode 1 also leaves them in
 // vfirst[t] (the first mixing layer of the model); vmode 2 stores (1 - lambda) v + lambda vfirst[t] (a later mixing layer; the
 // mixed values are what the cache keeps). grid (T, blocks): a warp per head, the heads and the value entries dealt over the blocks of a token.
@@ -170,6 +162,7 @@ struct GqaPrepArgs {
     const StepState * st;
     float * Q; float * cache; int ldc;
     float * vfirst; int vmode; float lambda;
+    int unit;
 };
 __global__ void __launch_bounds__(256) k_gqa_prep(const GqaPrepArgs a) {
     const int t = blockIdx.x, pos = a.st->pos0 + t, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -184,7 +177,7 @@ __global__ void __launch_bounds__(256) k_gqa_prep(const GqaPrepArgs a) {
         const float * w = is_q ? a.qw : a.kw;
         float * dst = is_q ? a.Q + (size_t) t * nq + (size_t) vec * a.D : row + (size_t) (vec - a.H) * a.D;
         float r = 1.0f;
-        if (w) {
+        if (w || a.unit) {
             float ss = 0.f;
             for (int i = lane; i < a.D; i += 32) ss = fmaf(src[i], src[i], ss);
             ss = warp_sum(ss);
@@ -192,12 +185,12 @@ __global__ void __launch_bounds__(256) k_gqa_prep(const GqaPrepArgs a) {
         }
         for (int i = lane; i < half; i += 32) {
             const int lo = rope_lo(a.rope, i), hi = rope_hi(a.rope, i);
-            const float x = w ? src[lo] * r * w[lo] : src[lo], y = w ? src[hi] * r * w[hi] : src[hi];
+            const float x = src[lo] * r * (w ? w[lo] : 1.0f), y = src[hi] * r * (w ? w[hi] : 1.0f);
             float ox, oy;
             rope_pair(a.rope, pos, i, x, y, ox, oy);
             dst[lo] = ox; dst[hi] = oy;
         }
-        for (int i = a.rope.dims + lane; i < a.D; i += 32) dst[i] = w ? src[i] * r * w[i] : src[i];
+        for (int i = a.rope.dims + lane; i < a.D; i += 32) dst[i] = src[i] * r * (w ? w[i] : 1.0f);
     }
     for (int i = bk * 256 + tid; i < nv; i += 256 * nblk) {
         float x = v[i];

@@ -1,6 +1,6 @@
 // stack_kernels_mix.cuh — more CUDA kernels (sm_100a) of the layer-stack models, beside stack_kernels.cuh: an element-wise
 // norm without statistics (dynamic tanh), the sub-layer join with a depth-weighted average over the outputs of all earlier
-// layers, retention (matrix state with a constant decay per head), sigmoid attention with a linear distance penalty over
+// layers, the rotation of retention (its recurrence is in stack_kernels_scan.cuh), sigmoid attention with a linear distance penalty over
 // grouped key/value heads, and the routed mixture of gated units (router with group-limited choice, expert-sorted rows for
 // the segmented products of prompt portions, indexed mat-vecs for single tokens).
 // Every size and constant is a kernel argument. Everything here is float32: norms, positions and angles, scores and
@@ -95,6 +95,129 @@ __global__ void __launch_bounds__(256) k_join(const JoinArgs a) {
     }
 }
 
+// ---- blocks whose sub-layers read the residual itself and are normed on the way out: X += mult * y / rms(y) * w ---------------------
+// y[t] is one of
+//   plain     Ya[t]
+//   pair      (Ya[t] / rms(Ya[t]) * wa + Yb[t] / rms(Yb[t]) * wb) / 2
+//   mixture   sum_k wt[t][k] y_k (+ sg[t] Ysh[t]): y_k is the chosen expert's output, Yk[slot(t, k)] (slot_of == nullptr: slot
+//             t top + k), or, for choices >= n_real (identity outputs), the sub-layer's input X[t] itself
+// and, after the model's last sub-layer, Hn[t] = X / rms(X) * fw (the head's input). One block per token; VEC-entry chunks of the row
+// are dealt over the threads, which keep POST_OWN of them in registers (rows beyond that go through `scratch`, [T][E]).
+struct PostJoinArgs {
+    float * X; int E; float eps, mult;
+    const float * w;                        // the norm's factors (1 + stored weight)
+    const float * Ya; const float * Yb; const float * wa; const float * wb;
+    const float * Yk; const float * wt; const int32_t * sel; const int32_t * slot_of; int top, n_real; const float * Ysh; const float * sg;
+    const float * fw; float * Hn;           // fw != nullptr: the model's norm
+    float * scratch;
+};
+constexpr int POST_OWN = 2;
+template <int NV> __device__ __forceinline__ void block_sums(float (&v)[NV], float (*red)[32]) {
+#pragma unroll
+    for (int i = 0; i < NV; i++) { v[i] = warp_sum(v[i]); if ((threadIdx.x & 31) == 0) red[i][threadIdx.x >> 5] = v[i]; }
+    __syncthreads();
+    const int nw = blockDim.x >> 5;
+#pragma unroll
+    for (int i = 0; i < NV; i++) { v[i] = 0.f; for (int w = 0; w < nw; w++) v[i] += red[i][w]; }
+    __syncthreads();
+}
+template <int VEC>
+__global__ void __launch_bounds__(1024) k_post_join(const PostJoinArgs a) {
+    __shared__ float red[2][32];
+    const int t = blockIdx.x, nt = blockDim.x, nchunk = a.E / VEC;
+    const size_t row = (size_t) t * a.E;
+    float ra = 1.f, rb = 1.f;
+    if (a.Yb) {
+        float s2[2] = { 0.f, 0.f };
+        for (int c = threadIdx.x; c < nchunk; c += nt) {
+            float u[VEC], v[VEC];
+            ld_chunk<VEC>(a.Ya + row + c * VEC, u); ld_chunk<VEC>(a.Yb + row + c * VEC, v);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) { s2[0] = fmaf(u[e], u[e], s2[0]); s2[1] = fmaf(v[e], v[e], s2[1]); }
+        }
+        block_sums<2>(s2, red);
+        ra = 0.5f / sqrtf(s2[0] / (float) a.E + a.eps); rb = 0.5f / sqrtf(s2[1] / (float) a.E + a.eps);
+    }
+    const float sg = a.Ysh ? a.sg[t] : 0.f;
+    float keep[POST_OWN][VEC], old[POST_OWN][VEC], ss[1] = { 0.f };
+    const auto output = [&](int i, const float (&x)[VEC], float (&y)[VEC]) {
+        if (a.Yk) {
+#pragma unroll
+            for (int e = 0; e < VEC; e++) y[e] = 0.f;
+            for (int k = 0; k < a.top; k++) {
+                const int s = t * a.top + k;
+                const float w = a.wt[s];
+                float v[VEC];
+                if (a.sel[s] >= a.n_real) {
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) v[e] = x[e];
+                } else ld_chunk<VEC>(a.Yk + (size_t) (a.slot_of ? a.slot_of[s] : s) * a.E + i, v);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) y[e] = fmaf(w, v[e], y[e]);
+            }
+            if (a.Ysh) {
+                float v[VEC];
+                ld_chunk<VEC>(a.Ysh + row + i, v);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) y[e] = fmaf(sg, v[e], y[e]);
+            }
+            return;
+        }
+        ld_chunk<VEC>(a.Ya + row + i, y);
+        if (a.Yb) {
+            float v[VEC], wa[VEC], wb[VEC];
+            ld_chunk<VEC>(a.Yb + row + i, v); ld_chunk<VEC>(a.wa + i, wa); ld_chunk<VEC>(a.wb + i, wb);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) y[e] = fmaf(y[e] * ra, wa[e], v[e] * rb * wb[e]);
+        }
+    };
+#pragma unroll
+    for (int k = 0; k < POST_OWN; k++) {
+        const int c = threadIdx.x + k * nt;
+        if (c < nchunk) {
+            ld_chunk<VEC>(a.X + row + c * VEC, old[k]);
+            output(c * VEC, old[k], keep[k]);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) ss[0] = fmaf(keep[k][e], keep[k][e], ss[0]);
+        }
+    }
+    for (int c = threadIdx.x + POST_OWN * nt; c < nchunk; c += nt) {
+        float x[VEC], y[VEC];
+        ld_chunk<VEC>(a.X + row + c * VEC, x);
+        output(c * VEC, x, y);
+        st_chunk<VEC>(a.scratch + row + c * VEC, y);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss[0] = fmaf(y[e], y[e], ss[0]);
+    }
+    block_sums<1>(ss, red);
+    const float r = 1.0f / sqrtf(ss[0] / (float) a.E + a.eps);
+    ss[0] = 0.f;
+    const auto finish = [&](int i, float (&x)[VEC], const float (&y)[VEC]) {
+        float w[VEC];
+        ld_chunk<VEC>(a.w + i, w);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) { x[e] = fmaf(a.mult, y[e] * r * w[e], x[e]); ss[0] = fmaf(x[e], x[e], ss[0]); }
+        st_chunk<VEC>(a.X + row + i, x);
+    };
+#pragma unroll
+    for (int k = 0; k < POST_OWN; k++) { const int c = threadIdx.x + k * nt; if (c < nchunk) finish(c * VEC, old[k], keep[k]); }
+    for (int c = threadIdx.x + POST_OWN * nt; c < nchunk; c += nt) {
+        float x[VEC], y[VEC];
+        ld_chunk<VEC>(a.X + row + c * VEC, x); ld_chunk<VEC>(a.scratch + row + c * VEC, y);
+        finish(c * VEC, x, y);
+    }
+    if (!a.fw) return;
+    block_sums<1>(ss, red);
+    const float f = 1.0f / sqrtf(ss[0] / (float) a.E + a.eps);
+    for (int c = threadIdx.x, k = 0; c < nchunk; c += nt, k++) {
+        float x[VEC], w[VEC];
+        ld_chunk<VEC>(a.X + row + c * VEC, x); ld_chunk<VEC>(a.fw + c * VEC, w);       // what this thread wrote
+#pragma unroll
+        for (int e = 0; e < VEC; e++) x[e] = x[e] * f * w[e];
+        st_chunk<VEC>(a.Hn + row + c * VEC, x);
+    }
+}
+
 // ---- retention: S <- decay_h S + k v^T, o = S^T q per head: a plain decayed sum, nothing divides the read-out --------------------------------------
 // P[t] = [ q: H x D | k: H x D | v: H x V | output-gate pre-activation: H x V ].
 // Step 1, per token, in place: the first rope.dims entries of every q and k head are rotated by the token's position
@@ -112,332 +235,7 @@ __global__ void k_retention_prep(float * __restrict__ P, int ldp, int q_off, int
         }
     }
 }
-// Step 2, the recurrence. S is [D][V] per head in float32 and stays in registers for the whole portion; four neighbouring lanes
-// share one column of S, each holding a quarter of its rows, and close the read-out with two shuffles. q and k of a few tokens
-// arrive in shared memory by asynchronous copies while the tokens before them are walked (two buffers); each quarter of the rows
-// is padded apart so that the four lanes' reads fall into different banks. A head's columns are spread over gridDim.y blocks.
-template <int DMAX>
-__global__ void __launch_bounds__(512) k_retention_scan(const float * __restrict__ P, int ldp, int q_off, int k_off, int v_off, const float * __restrict__ decay,
-                                                        int T, int H, int D, int V, float * __restrict__ S, float * __restrict__ O) {
-    constexpr int TT = DMAX > 128 ? 4 : 8, DR = DMAX / GD_RG, ROW = GD_RG * (DR + GD_PAD);
-    __shared__ __align__(16) float qs[2][TT][ROW], ks[2][TT][ROW], vs[2][TT][128];
-    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, rg = lane & 3, ncols = blockDim.x / GD_RG;
-    const int cl = (tid >> 5) * 8 + (lane >> 2), col = blockIdx.y * ncols + cl;
-    const bool live = col < V;
-    const float g = decay[h];
-    const auto stage = [&](int t0, int buf) {
-        const int nt = min(TT, T - t0);
-        for (int i = tid; i < nt * DMAX; i += blockDim.x) {
-            const int tt = i / DMAX, d = i % DMAX, at = (d / DR) * (DR + GD_PAD) + d % DR;
-            const bool in = d < D;
-            const float * p = P + (size_t) (t0 + tt) * ldp + (size_t) h * D + (in ? d : 0);
-            cp_async4(&qs[buf][tt][at], p + q_off, in);
-            cp_async4(&ks[buf][tt][at], p + k_off, in);
-        }
-        for (int i = tid; i < nt * ncols; i += blockDim.x) {
-            const int tt = i / ncols, c = i % ncols;
-            const bool in = blockIdx.y * ncols + c < V;
-            cp_async4(&vs[buf][tt][c], P + (size_t) (t0 + tt) * ldp + v_off + (size_t) h * V + (in ? blockIdx.y * ncols + c : 0), in);
-        }
-    };
-    stage(0, 0);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    float s[DR];
-    float * Sh = S + (size_t) h * D * V;
-#pragma unroll
-    for (int i = 0; i < DR; i++) { const int d = rg * DR + i; s[i] = (live && d < D) ? Sh[(size_t) d * V + col] : 0.f; }
-    const int base = rg * (DR + GD_PAD);
-    for (int t0 = 0, buf = 0; t0 < T; t0 += TT, buf ^= 1) {
-        const int nt = min(TT, T - t0);
-        if (t0 + TT < T) stage(t0 + TT, buf ^ 1);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();
-        for (int tt = 0; tt < nt; tt++) {
-            const float v = vs[buf][tt][cl];
-            float op[4] = { 0.f, 0.f, 0.f, 0.f };
-#pragma unroll
-            for (int i = 0; i < DR; i++) {
-                s[i] = fmaf(g, s[i], ks[buf][tt][base + i] * v);
-                op[i & 3] = fmaf(s[i], qs[buf][tt][base + i], op[i & 3]);
-            }
-            float o = (op[0] + op[1]) + (op[2] + op[3]);
-            o += __shfl_xor_sync(0xffffffffu, o, 1);
-            o += __shfl_xor_sync(0xffffffffu, o, 2);
-            if (rg == 0 && live) O[(size_t) (t0 + tt) * H * V + (size_t) h * V + col] = o;
-        }
-        __syncthreads();
-    }
-    if (live) {
-#pragma unroll
-        for (int i = 0; i < DR; i++) { const int d = rg * DR + i; if (d < D) Sh[(size_t) d * V + col] = s[i]; }
-    }
-}
-
-// Long prompt portions run the same recurrence chunk by chunk (RC tokens), so that only the short walk over chunks is serial.
-// With t, j local to chunk c of n_c tokens, S_c the state before it and g the head's decay:
-//   U_c = sum_j g^(n_c - 1 - j) k_j v_j^T                               k_retention_chunk_kv     (all chunks at once)
-//   S_(c+1) = g^(n_c) S_c + U_c                                         k_retention_chunk_state  (in place: U_c's slot then holds S_c)
-//   o_t = g^(t + 1) S_c^T q_t + sum_(j <= t) g^(t - j) (q_t . k_j) v_j  k_retention_chunk_out    (all chunks at once)
-// Same float32 arithmetic as the walk, sums in another order. SB [H][chunks][D][V] is a working buffer of the pass.
-constexpr int RC = 32;
-// rows [0, n_rows) x columns [0, n_cols) of a row-major source into a shared tile of `rows` x `cols` (row stride dst_ld), zeros
-// elsewhere, by asynchronous copies that are all issued before any is awaited (16 bytes each when `vec`: every address a multiple of 16)
-__device__ __forceinline__ void stage_tile_async(float * dst, int dst_ld, const float * src, size_t src_ld, int rows, int cols, int n_rows, int n_cols, bool vec, int tid, int nthreads) {
-    if (vec) {
-        const int c4 = cols >> 2;
-        for (int i = tid; i < rows * c4; i += nthreads) {
-            const int j = i / c4, x = (i - j * c4) << 2;
-            const bool in = j < n_rows && x < n_cols;
-            cp_async16((uint32_t) __cvta_generic_to_shared(dst + j * dst_ld + x), in ? (const void *) (src + (size_t) j * src_ld + x) : (const void *) src, in ? 16u : 0u);
-        }
-    } else {
-        for (int i = tid; i < rows * cols; i += nthreads) {
-            const int j = i / cols, x = i - j * cols;
-            const bool in = j < n_rows && x < n_cols;
-            cp_async4(dst + j * dst_ld + x, in ? src + (size_t) j * src_ld + x : src, in);
-        }
-    }
-}
-__device__ __forceinline__ void async_copies_done() {
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-}
-// grid (H, chunks, ceil(V / 128)), 256 threads: thread (ty, tx) owns 8 x 8 of a 128 x 128 tile of U_c; keys and decay-scaled values
-// of the chunk are staged in shared memory
-__global__ void __launch_bounds__(256) k_retention_chunk_kv(const float * __restrict__ P, int ldp, int k_off, int v_off, const float * __restrict__ decay,
-                                                            int T, int H, int D, int V, float * __restrict__ SB) {
-    __shared__ __align__(16) float Ks[RC][128], Vs[RC][128];
-    const int h = blockIdx.x, c = blockIdx.y, v0 = blockIdx.z * 128, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const int t0 = c * RC, nt = min(RC, T - t0), nch = gridDim.y;
-    __shared__ float pw[RC];
-    const float g = decay[h];
-    const bool vec = ((ldp | k_off | v_off | D | V) & 3) == 0;
-    if (tid < RC) pw[tid] = tid < nt ? powf(g, (float) (nt - 1 - tid)) : 0.f;
-    stage_tile_async(&Vs[0][0], 128, P + (size_t) t0 * ldp + v_off + (size_t) h * V + v0, (size_t) ldp, RC, 128, nt, V - v0, vec, tid, 256);
-    float * U = SB + ((size_t) h * nch + c) * D * V;
-    for (int d0 = 0; d0 < D; d0 += 128) {
-        __syncthreads();
-        stage_tile_async(&Ks[0][0], 128, P + (size_t) t0 * ldp + k_off + (size_t) h * D + d0, (size_t) ldp, RC, 128, nt, D - d0, vec, tid, 256);
-        async_copies_done();
-        __syncthreads();
-        float acc[8][8];
-#pragma unroll
-        for (int a = 0; a < 8; a++)
-#pragma unroll
-            for (int b = 0; b < 8; b++) acc[a][b] = 0.f;
-#pragma unroll 4
-        for (int j = 0; j < RC; j++) {
-            const float4 ka = *reinterpret_cast<const float4 *>(&Ks[j][ty * 8]), kb = *reinterpret_cast<const float4 *>(&Ks[j][ty * 8 + 4]);
-            const float4 va = *reinterpret_cast<const float4 *>(&Vs[j][tx * 8]), vb = *reinterpret_cast<const float4 *>(&Vs[j][tx * 8 + 4]);
-            const float f = pw[j];                      // the key's decay until the chunk's end
-            const float kk[8] = { ka.x * f, ka.y * f, ka.z * f, ka.w * f, kb.x * f, kb.y * f, kb.z * f, kb.w * f }, vv[8] = { va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w };
-#pragma unroll
-            for (int a = 0; a < 8; a++)
-#pragma unroll
-                for (int b = 0; b < 8; b++) acc[a][b] = fmaf(kk[a], vv[b], acc[a][b]);
-        }
-#pragma unroll
-        for (int a = 0; a < 8; a++) {
-            const int d = d0 + ty * 8 + a;
-            if (d >= D) continue;
-#pragma unroll
-            for (int b = 0; b < 8; b++) { const int v = v0 + tx * 8 + b; if (v < V) U[(size_t) d * V + v] = acc[a][b]; }
-        }
-    }
-}
-// grid (H, ceil(D V / 256)): a thread owns one entry of the state and walks the chunks
-__global__ void k_retention_chunk_state(const float * __restrict__ decay, int T, int D, int V, int nch, float * __restrict__ S, float * __restrict__ SB) {
-    const int h = blockIdx.x, e = blockIdx.y * blockDim.x + threadIdx.x, n = D * V;
-    if (e >= n) return;
-    const float g = decay[h], gfull = powf(g, (float) RC), glast = powf(g, (float) (T - (nch - 1) * RC));
-    float s = S[(size_t) h * n + e];
-    float * sb = SB + (size_t) h * nch * n + e;
-    for (int c0 = 0; c0 < nch; c0 += 8) {
-        float u[8];
-#pragma unroll
-        for (int i = 0; i < 8; i++) u[i] = c0 + i < nch ? sb[(size_t) (c0 + i) * n] : 0.f;
-#pragma unroll
-        for (int i = 0; i < 8; i++) {
-            if (c0 + i < nch) {
-                sb[(size_t) (c0 + i) * n] = s;
-                s = fmaf(c0 + i == nch - 1 ? glast : gfull, s, u[i]);
-            }
-        }
-    }
-    S[(size_t) h * n + e] = s;
-}
-// grid (H, chunks, ceil(V / 128)), 128 threads: warp w owns tokens 8 w .. 8 w + 7 of the chunk, a lane four value channels.
-// Dynamic shared memory: q and k of the chunk [RC][D + 4] each, the masked scores [RC][RC + 4], the values [RC][128], the powers of g.
-__global__ void __launch_bounds__(128) k_retention_chunk_out(const float * __restrict__ P, int ldp, int q_off, int k_off, int v_off, const float * __restrict__ decay,
-                                                             int T, int H, int D, int V, const float * __restrict__ SB, float * __restrict__ O) {
-    extern __shared__ __align__(16) float csm[];
-    const int Dp = D + 4;
-    constexpr int AP = RC + 4;                         // score rows padded to whole 16-byte chunks
-    float * Qs = csm, * Ks = Qs + RC * Dp, * As = Ks + RC * Dp, * Vs = As + RC * AP, * pw = Vs + RC * 128;
-    const int h = blockIdx.x, c = blockIdx.y, v0 = blockIdx.z * 128, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int t0 = c * RC, nt = min(RC, T - t0), nch = gridDim.y;
-    const float g = decay[h];
-    {
-        const bool al = ((ldp | q_off | k_off | v_off | D | V) & 3) == 0;
-        const float * row0 = P + (size_t) t0 * ldp + (size_t) h * D;
-        stage_tile_async(Qs, Dp, row0 + q_off, (size_t) ldp, RC, D, nt, D, al, tid, 128);
-        stage_tile_async(Ks, Dp, row0 + k_off, (size_t) ldp, RC, D, nt, D, al, tid, 128);
-        stage_tile_async(Vs, 128, P + (size_t) t0 * ldp + v_off + (size_t) h * V + v0, (size_t) ldp, RC, 128, nt, V - v0, al, tid, 128);
-        if (tid <= RC) pw[tid] = powf(g, (float) tid);
-        async_copies_done();
-    }
-    __syncthreads();
-    const int D4 = (D & 3) ? 0 : D;                    // 16-byte reads along d need whole chunks per row (D + 4 is then a multiple of 4 too)
-    {   // scores of the chunk against itself: lane = key j, the warp's 8 tokens; 16-byte reads along d (a lane's own key row, the
-        // tokens' query rows as broadcasts) when D is a multiple of 4, else entry by entry
-        float sc[8] = { 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f };
-        const float * kr = Ks + lane * Dp;
-        for (int d = 0; d < D4; d += 4) {
-            const float4 k4 = *reinterpret_cast<const float4 *>(kr + d);
-#pragma unroll
-            for (int a = 0; a < 8; a++) {
-                const float4 q4 = *reinterpret_cast<const float4 *>(Qs + (warp * 8 + a) * Dp + d);
-                sc[a] = fmaf(q4.x, k4.x, fmaf(q4.y, k4.y, fmaf(q4.z, k4.z, fmaf(q4.w, k4.w, sc[a]))));
-            }
-        }
-        for (int d = D4; d < D; d++)
-#pragma unroll
-            for (int a = 0; a < 8; a++) sc[a] = fmaf(Qs[(warp * 8 + a) * Dp + d], kr[d], sc[a]);
-#pragma unroll
-        for (int a = 0; a < 8; a++) { const int t = warp * 8 + a; As[t * AP + lane] = lane <= t ? sc[a] * pw[t - lane] : 0.f; }
-    }
-    __syncthreads();
-    float acc[8][4];
-#pragma unroll
-    for (int a = 0; a < 8; a++)
-#pragma unroll
-        for (int b = 0; b < 4; b++) acc[a][b] = 0.f;
-    const float * Sc = SB + ((size_t) h * nch + c) * D * V;
-    const int v = v0 + lane * 4;
-    const bool vec = (V & 3) == 0 && v + 3 < V;
-    const auto srow = [&](int d, float (&sv)[4]) {
-        if (vec) { const float4 f = __ldg(reinterpret_cast<const float4 *>(Sc + (size_t) d * V + v)); sv[0] = f.x; sv[1] = f.y; sv[2] = f.z; sv[3] = f.w; }
-        else {
-#pragma unroll
-            for (int b = 0; b < 4; b++) sv[b] = v + b < V ? __ldg(Sc + (size_t) d * V + v + b) : 0.f;
-        }
-    };
-#pragma unroll 2
-    for (int d = 0; d < D4; d += 4) {                   // four rows of the chunk's entry state per step, the queries as 16-byte broadcasts
-        float sv[4][4];
-#pragma unroll
-        for (int r = 0; r < 4; r++) srow(d + r, sv[r]);
-#pragma unroll
-        for (int a = 0; a < 8; a++) {
-            const float4 q4 = *reinterpret_cast<const float4 *>(Qs + (warp * 8 + a) * Dp + d);
-#pragma unroll
-            for (int b = 0; b < 4; b++) acc[a][b] = fmaf(q4.x, sv[0][b], fmaf(q4.y, sv[1][b], fmaf(q4.z, sv[2][b], fmaf(q4.w, sv[3][b], acc[a][b]))));
-        }
-    }
-    for (int d = D4; d < D; d++) {
-        float sv[4];
-        srow(d, sv);
-#pragma unroll
-        for (int a = 0; a < 8; a++) {
-            const float qv = Qs[(warp * 8 + a) * Dp + d];
-#pragma unroll
-            for (int b = 0; b < 4; b++) acc[a][b] = fmaf(qv, sv[b], acc[a][b]);
-        }
-    }
-#pragma unroll
-    for (int a = 0; a < 8; a++) {
-        const float f = pw[warp * 8 + a + 1];
-#pragma unroll
-        for (int b = 0; b < 4; b++) acc[a][b] *= f;
-    }
-    for (int j = 0; j < RC; j += 4) {
-        float4 f[4];
-#pragma unroll
-        for (int r = 0; r < 4; r++) f[r] = *reinterpret_cast<const float4 *>(Vs + (j + r) * 128 + lane * 4);
-#pragma unroll
-        for (int a = 0; a < 8; a++) {
-            const float4 w = *reinterpret_cast<const float4 *>(As + (warp * 8 + a) * AP + j);
-            acc[a][0] = fmaf(w.x, f[0].x, fmaf(w.y, f[1].x, fmaf(w.z, f[2].x, fmaf(w.w, f[3].x, acc[a][0]))));
-            acc[a][1] = fmaf(w.x, f[0].y, fmaf(w.y, f[1].y, fmaf(w.z, f[2].y, fmaf(w.w, f[3].y, acc[a][1]))));
-            acc[a][2] = fmaf(w.x, f[0].z, fmaf(w.y, f[1].z, fmaf(w.z, f[2].z, fmaf(w.w, f[3].z, acc[a][2]))));
-            acc[a][3] = fmaf(w.x, f[0].w, fmaf(w.y, f[1].w, fmaf(w.z, f[2].w, fmaf(w.w, f[3].w, acc[a][3]))));
-        }
-    }
-#pragma unroll
-    for (int a = 0; a < 8; a++) {
-        const int tl = warp * 8 + a;
-        if (tl >= nt) continue;
-#pragma unroll
-        for (int b = 0; b < 4; b++) if (v + b < V) O[(size_t) (t0 + tl) * H * V + (size_t) h * V + v + b] = acc[a][b];
-    }
-}
-
-// The whole mixer core for a one-token step in one launch (steps 1 and 2 and the read-out's norm and gate): one block per head.
-// Rotation and key scale happen on the way into shared memory, the state is updated tile by tile of up to 128 columns (the same
-// four-lanes-per-column layout), the head's read-out is kept in shared memory, then A[h] = o / rms(o) * silu(gate) (eps inside the
-// root, no weight). Dynamic shared memory: V floats.
-template <int DMAX>
-__global__ void __launch_bounds__(512) k_retention_token(const float * __restrict__ P, int q_off, int k_off, int v_off, int g_off, const float * __restrict__ decay,
-                                                         RopeArgs rope, float k_scale, const StepState * __restrict__ st, int H, int D, int V, float eps,
-                                                         float * __restrict__ S, float * __restrict__ A) {
-    constexpr int DR = DMAX / GD_RG, ROW = GD_RG * (DR + GD_PAD);
-    extern __shared__ float o_s[];                      // [V]
-    __shared__ __align__(16) float qs[ROW], ks[ROW];
-    __shared__ float red[16];
-    const int h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rg = lane & 3, ncols = blockDim.x / GD_RG;
-    const int pos = st->pos0, half = rope.dims / 2;
-    const float * q = P + q_off + (size_t) h * D, * k = P + k_off + (size_t) h * D;
-    for (int i = tid; i < 2 * DMAX; i += blockDim.x) {
-        const bool is_k = i >= DMAX;
-        const int d = is_k ? i - DMAX : i, at = (d / DR) * (DR + GD_PAD) + d % DR;
-        float v = 0.f;
-        if (d < D) {
-            const float * x = is_k ? k : q;
-            if (d < half) { float a, b; rope_pair(rope, pos, d, x[d], x[d + half], a, b); v = a; }
-            else if (d < rope.dims) { float a, b; rope_pair(rope, pos, d - half, x[d - half], x[d], a, b); v = b; }
-            else v = x[d];
-            if (is_k) v *= k_scale;
-        }
-        (is_k ? ks : qs)[at] = v;
-    }
-    __syncthreads();
-    const float g = decay[h];
-    float * Sh = S + (size_t) h * D * V;
-    const int base = rg * (DR + GD_PAD), cl = warp * 8 + (lane >> 2);
-    float ss = 0.f;
-    for (int c0 = 0; c0 < V; c0 += ncols) {
-        const int col = c0 + cl;
-        const bool live = col < V;
-        const float v = live ? P[v_off + (size_t) h * V + col] : 0.f;
-        float op[4] = { 0.f, 0.f, 0.f, 0.f };
-        constexpr int CH = DR < 16 ? DR : 16;           // rows whose loads are in flight together (the stores would order them otherwise)
-#pragma unroll 1
-        for (int i0 = 0; i0 < DR; i0 += CH) {
-            float sv[CH];
-#pragma unroll
-            for (int i = 0; i < CH; i++) { const int d = rg * DR + i0 + i; sv[i] = (live && d < D) ? Sh[(size_t) d * V + col] : 0.f; }
-#pragma unroll
-            for (int i = 0; i < CH; i++) {
-                const int d = rg * DR + i0 + i;
-                sv[i] = fmaf(g, sv[i], ks[base + i0 + i] * v);
-                if (live && d < D) Sh[(size_t) d * V + col] = sv[i];
-                op[i & 3] = fmaf(sv[i], qs[base + i0 + i], op[i & 3]);
-            }
-        }
-        float o = (op[0] + op[1]) + (op[2] + op[3]);
-        o += __shfl_xor_sync(0xffffffffu, o, 1);
-        o += __shfl_xor_sync(0xffffffffu, o, 2);
-        if (rg == 0 && live) { o_s[col] = o; ss = fmaf(o, o, ss); }
-    }
-    ss = warp_sum(ss);
-    if (lane == 0) red[warp] = ss;
-    __syncthreads();
-    float tot = 0.f;
-    for (int w = 0; w < (int) (blockDim.x >> 5); w++) tot += red[w];
-    const float r = 1.0f / sqrtf(tot / (float) V + eps);
-    for (int i = tid; i < V; i += blockDim.x) A[(size_t) h * V + i] = o_s[i] * r * siluf_(P[g_off + (size_t) h * V + i]);
-}
+// Step 2 is the decayed outer-product recurrence of stack_kernels_scan.cuh with one constant decay per head.
 
 // ---- sigmoid attention over grouped key/value heads -------------------------------------------------------------------------------
 // P[t] = [ q: H x D | k: G x D | v: G x V ]. Query head h reads key/value head h / (H / G); position p sees every j <= p.
@@ -617,9 +415,10 @@ __global__ void k_group_o_layout(const float * __restrict__ Or, int Tpad, int H,
 
 // ---- routed mixture of gated units --------------------------------------------------------------------------------------------------
 // Router, per token, in float32: z = W_r h, s = softmax(z) over all n experts (score_fn 0) or s_i = sigmoid(z_i), each expert by
-// itself (score_fn 1). The expert list is cut into n_groups consecutive blocks
-// of equal size; a block ranks by the best s inside it and the choice is confined to the `keep` best-ranked blocks: of their experts
-// the `top` with the largest s are taken (lowest index first among equals), each weighing in with s * scale as it is.
+// itself (score_fn 1). Choices go by c = s + corr (corr == nullptr: c = s). The expert list is cut into n_groups consecutive blocks
+// of equal size; a block ranks by the best c inside it and the choice is confined to the `keep` best-ranked blocks: of their experts
+// the `top` with the largest c are taken (lowest index first among equals). A choice weighs in with s * scale as it is, or, with
+// `norm_w`, with s * scale over the sum of the chosen s (+ 1e-20).
 // sel[t][top], wt[t][top]; sg[t] = sigmoid(w_sg . h) is the shared unit's gate (w_sg == nullptr: no shared unit).
 // grid (T, ceil(rows / (8 / wpr))) with rows = n (+ 1 for the shared gate): wpr warps per row of the router (1, or 8 for steps of few
 // tokens, whose rows would otherwise be walked by one warp each), several 16-byte loads in flight;
@@ -634,6 +433,8 @@ struct RouteArgs {
     float * z; int * counter;
     int score_fn;       // 0: soft-max over the experts; 1: sigmoid of each logit
     int wpr;            // warps per router row: 1 (a block takes 8 rows) or 8 (a block takes one row, each warp an eighth of it: steps of few tokens)
+    const float * corr = nullptr;
+    int norm_w = 0;
 };
 __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
     extern __shared__ float rsm[];
@@ -678,7 +479,7 @@ __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
     if (warp != 0) return;
     const int per = a.n / a.n_groups;
     if (a.score_fn == 1) {
-        for (int i = lane; i < a.n; i += 32) { s[i] = sigmoidf_(__ldcg(z + i)); elig[i] = -1.f; }
+        for (int i = lane; i < a.n; i += 32) { s[i] = sigmoidf_(__ldcg(z + i)); elig[i] = -INFINITY; }
     } else {
         float mx = -INFINITY;
         for (int i = lane; i < a.n; i += 32) { const float v = __ldcg(z + i); s[i] = v; mx = fmaxf(mx, v); }
@@ -687,39 +488,46 @@ __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
         for (int i = lane; i < a.n; i += 32) { const float v = expf(s[i] - mx); s[i] = v; sum += v; }
         sum = warp_sum(sum);
         const float inv = 1.0f / sum;
-        for (int i = lane; i < a.n; i += 32) { s[i] *= inv; elig[i] = -1.f; }
+        for (int i = lane; i < a.n; i += 32) { s[i] *= inv; elig[i] = -INFINITY; }
     }
     __syncwarp();
     for (int g = lane; g < a.n_groups; g += 32) {
-        float b = -1.f;
-        for (int i = 0; i < per; i++) b = fmaxf(b, s[g * per + i]);
+        float b = -INFINITY;
+        for (int i = 0; i < per; i++) b = fmaxf(b, s[g * per + i] + (a.corr ? a.corr[g * per + i] : 0.f));
         gbest[g] = b;
     }
     __syncwarp();
     // the best groups, one at a time; then the best eligible experts, one at a time (value, then lowest index)
     for (int r = 0; r < a.keep; r++) {
-        float bv = -2.f; int bi = 0x7fffffff;
+        float bv = -INFINITY; int bi = 0x7fffffff;
         for (int g = lane; g < a.n_groups; g += 32) if (gbest[g] > bv) { bv = gbest[g]; bi = g; }
         for (int o = 16; o > 0; o >>= 1) {
             const float ov = __shfl_xor_sync(0xffffffffu, bv, o); const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
         if (bi != 0x7fffffff) {
-            for (int i = lane; i < per; i += 32) elig[bi * per + i] = s[bi * per + i];
-            if (lane == 0) gbest[bi] = -3.f;
+            for (int i = lane; i < per; i += 32) elig[bi * per + i] = s[bi * per + i] + (a.corr ? a.corr[bi * per + i] : 0.f);
+            if (lane == 0) gbest[bi] = -INFINITY;
         }
         __syncwarp();
     }
+    float chosen = 0.f;
     for (int r = 0; r < a.top; r++) {
-        float bv = -0.5f; int bi = 0x7fffffff;
+        float bv = -INFINITY; int bi = 0x7fffffff;
         for (int i = lane; i < a.n; i += 32) if (elig[i] > bv) { bv = elig[i]; bi = i; }
         for (int o = 16; o > 0; o >>= 1) {
             const float ov = __shfl_xor_sync(0xffffffffu, bv, o); const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
-        if (bi == 0x7fffffff) { bi = 0; bv = 0.f; }        // fewer eligible experts than `top` (refused at load): a slot of weight 0
-        if (lane == 0) { a.sel[t * a.top + r] = bi; a.wt[t * a.top + r] = bv * a.scale; elig[bi] = -1.f; }
+        const float w = bi == 0x7fffffff ? 0.f : s[bi];    // none left: fewer eligible experts than `top` (refused at load), or a score that is no number: a slot of weight 0
+        if (bi == 0x7fffffff) bi = 0;
+        chosen += w;
+        if (lane == 0) { a.sel[t * a.top + r] = bi; a.wt[t * a.top + r] = w * a.scale; elig[bi] = -INFINITY; }
         __syncwarp();
+    }
+    if (a.norm_w) {
+        const float f = 1.0f / (chosen + 1e-20f);
+        for (int r = lane; r < a.top; r += 32) a.wt[t * a.top + r] *= f;
     }
 }
 // Prompt portions: the n_slots = T top (token, choice) slots sorted by expert, stably, so that every expert's rows are contiguous:
