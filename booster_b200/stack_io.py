@@ -1,4 +1,4 @@
-"""Synthetic models of the layer-stack family (Matulorn, Dopilorn, Tosevik and Rumurax designs; config.json + model.safetensors) for benchmarks and smoke runs: random
+"""Synthetic models of the layer-stack family (Matulorn, Dopilorn, Tosevik, Rumurax and Kogerax designs; config.json + model.safetensors) for benchmarks and smoke runs: random
 bfloat16 weights of the right shapes, the counterpart of gguf_io.synth_llama for the GGUF path. Pure host code."""
 from __future__ import annotations
 
@@ -100,6 +100,31 @@ def rumurax_config(width: int, n_layer: int, ff: int, heads: int, vocab: int = 3
     return {"architecture": "Rumurax", "layers": layers, "norm": {"eps": 1e-6}, "streams": streams, "vocab": vocab, "width": width}
 
 
+def kogerax_config(width: int, n_layer: int, ff: int, heads: int, vocab: int = 32000, head_dim: int = 128, kv_heads: int = 0, experts: int = 16, top: int = 4,
+                   identity: int = 2, window: int = 1024, state: int = 128, scan_state: int = 16, expand: int = 2, ssd_head: int = 64,
+                   pattern=("parallel", "mlstm", "mamba2")) -> dict:
+    """a Kogerax configuration whose layers resemble a real model's: mixers in `pattern` order, a dense feed-forward on the first layer, on
+    the others a routed mixture whose chosen experts plus the shared unit are as wide together as a dense feed-forward of `ff`
+    (top x 3 ff / 16 + ff / 4)"""
+    e_ff = max(8, ff * 3 // (4 * top) // 8 * 8)
+    inner = expand * width
+    layers = []
+    for i in range(n_layer):
+        kind = pattern[i % len(pattern)]
+        if kind == "parallel":
+            mx = {"left": {"heads": heads, "kv_heads": kv_heads or max(1, heads // 4), "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "mask": {"size": window},
+                           "rot": {"base": 500000.0, "dims": head_dim // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+                  "right": {"inner": inner, "state": scan_state, "dt_rank": max(1, width // 16), "conv": 4}}
+        elif kind == "mlstm":
+            mx = {"heads": heads, "dim": head_dim, "vdim": head_dim, "gate_cap": 15.0}
+        else:
+            mx = {"heads": inner // ssd_head, "vdim": ssd_head, "state": state, "groups": 1, "norm_groups": 1, "conv": 4}
+        mlp = {"kind": "dense", "ff": ff} if i == 0 else {"kind": "moe", "expert": {"ff": e_ff, "limit": 7.0}, "shared": {"ff": ff - top * e_ff, "limit": 7.0},
+                                                          "router": {"experts": experts, "identity": identity, "top": top}}
+        layers.append({"type": kind, "mixer": mx, "mlp": mlp})
+    return {"architecture": "Kogerax", "embedding": {"scale": float(width) ** 0.5}, "layers": layers, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": vocab, "width": width}
+
+
 def rumurax_shapes(cfg: dict) -> Dict[str, List[int]]:
     E, V, S = cfg["width"], cfg["vocab"], cfg.get("streams", 1)
     t: Dict[str, List[int]] = {"embed": [V, E]}
@@ -130,6 +155,48 @@ def rumurax_shapes(cfg: dict) -> Dict[str, List[int]]:
                 t.update({p + "mlp." + u + "gate": [f, E], p + "mlp." + u + "up": [f, E], p + "mlp." + u + "down": [E, f]})
             t[p + "mlp.router"] = [mj["router"]["experts"], E]
     t["final.norm"] = []
+    t["head"] = [V, E]
+    return t
+
+
+def kogerax_shapes(cfg: dict) -> Dict[str, List[int]]:
+    E, V = cfg["width"], cfg["vocab"]
+    t: Dict[str, List[int]] = {"embed": [V, E]}
+    for i, L in enumerate(cfg["layers"]):
+        p, mx = f"l{i}.", L["mixer"]
+        m = p + "mix."
+        t[p + "norm1"] = [E]
+        if L["type"] == "parallel":
+            a, s = mx["left"], mx["right"]
+            H, G, D, Vd = a["heads"], a.get("kv_heads", a["heads"]), a["dim"], a["vdim"]
+            n, N, R = s["inner"], s["state"], s["dt_rank"]
+            t.update({m + "left.q": [H * D, E], m + "left.k": [G * D, E], m + "left.v": [G * Vd, E], m + "left.o": [E, H * Vd], m + "left.out": [E],
+                      m + "right.in": [2 * n, E], m + "right.conv": [n, s["conv"]], m + "right.conv.b": [n], m + "right.x": [R + 2 * N, n], m + "right.dt": [n, R],
+                      m + "right.dt.b": [n], m + "right.A_log": [n, N], m + "right.D": [n], m + "right.o": [E, n], m + "right.out": [E]})
+        elif L["type"] == "mlstm":
+            H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
+            t.update({m + "q": [H * D, E], m + "k": [H * D, E], m + "v": [H * Vd, E], m + "g": [H * Vd, E], m + "i": [H, E], m + "i.b": [H], m + "f": [H, E], m + "f.b": [H],
+                      m + "norm": [H * Vd], m + "o": [E, H * Vd]})
+        elif L["type"] == "mamba2":
+            H, inner, gn = mx["heads"], mx["heads"] * mx["vdim"], mx["groups"] * mx["state"]
+            t.update({m + "in": [2 * inner + 2 * gn + H, E], m + "conv": [inner + 2 * gn, mx["conv"]], m + "conv.b": [inner + 2 * gn], m + "dt_bias": [H], m + "A_log": [H], m + "D": [H],
+                      m + "norm": [inner], m + "o": [E, inner]})
+        else:
+            raise ValueError(L["type"])
+        mj = L.get("mlp")
+        if not mj:
+            continue
+        t[p + "norm2"] = [E]
+        units = [("", mj["ff"])] if mj["kind"] == "dense" else [(f"e{e}.", mj["expert"]["ff"]) for e in range(mj["router"]["experts"])]
+        if mj["kind"] != "dense":
+            rows = mj["router"]["experts"] + mj["router"].get("identity", 0)
+            t.update({p + "mlp.router": [rows, E], p + "mlp.correction": [rows]})
+            if mj.get("shared"):
+                units.append(("shared.", mj["shared"]["ff"]))
+                t[p + "mlp.shared.sg"] = [1, E]
+        for u, f in units:
+            t.update({p + "mlp." + u + "gate": [f, E], p + "mlp." + u + "up": [f, E], p + "mlp." + u + "down": [E, f]})
+    t["final.norm"] = [E]
     t["head"] = [V, E]
     return t
 
@@ -227,6 +294,8 @@ def tensor_shapes(cfg: dict) -> Dict[str, List[int]]:
         return tosevik_shapes(cfg)
     if cfg.get("architecture") == "Rumurax":
         return rumurax_shapes(cfg)
+    if cfg.get("architecture") == "Kogerax":
+        return kogerax_shapes(cfg)
     E, V = cfg["width"], cfg["vocab"]
     t = {"embed": [V, E]}
     for i, L in enumerate(cfg["layers"]):
@@ -273,8 +342,8 @@ def synth_stack(d: str, cfg: dict, seed: int = 1234) -> str:
         f.write(hj)
         for name, shp in shapes.items():
             n = int(np.prod(shp))
-            zero_centred = cfg.get("architecture") == "Dopilorn" and name.rsplit(".", 1)[-1] in ("norm1", "norm2") or name == "final.norm" and cfg.get("architecture") == "Dopilorn"
             leaf = name.rsplit(".", 1)[-1]
+            zero_centred = cfg.get("architecture") in ("Dopilorn", "Kogerax") and (leaf in ("norm1", "norm2") or name == "final.norm")
             if cfg.get("architecture") == "Tosevik" and leaf in ("b", "alpha", "dwa", "pb"):
                 if leaf == "dwa":                                # mostly the layer's own result, a little of every earlier one
                     x = (0.3 / math.sqrt(n)) * rng.standard_normal(n, dtype=np.float32)
@@ -294,6 +363,8 @@ def synth_stack(d: str, cfg: dict, seed: int = 1234) -> str:
                     x = np.full(1, 0.5, np.float32)
                 else:                                            # positive: the penalty is r1 ln(1 + r2 distance)
                     x = 0.1 + rng.random(n, dtype=np.float32)
+            elif cfg.get("architecture") == "Kogerax" and (leaf in ("correction", "out", "D", "dt_bias") or name.endswith((".f.b", ".dt.b"))):
+                x = {"correction": 0.0, "out": 1.0, "D": 1.0, "dt_bias": -3.0}.get(leaf, 3.0 if name.endswith(".f.b") else -3.0) + 0.05 * rng.standard_normal(n, dtype=np.float32)
             elif name.endswith("mlp.act"):
                 x = np.array([1.0, 0.5, 0.25, 0.0], np.float32)
             elif "canon" in name or zero_centred or name == "loop.step":

@@ -129,6 +129,10 @@ def parallel(h, mx, W, p, eps):
     return 0.5 * (rms_unit(a, eps) * W[p + "left.out"] + rms_unit(b, eps) * W[p + "right.out"])
 
 
+def divisor(nq, m):
+    return max(abs(nq), np.exp(-m)) + 1e-6
+
+
 def mlstm(h, mx, W, p, eps):
     T = h.shape[0]
     H, D, V, cap = mx["heads"], mx["dim"], mx["vdim"], mx["gate_cap"]
@@ -146,7 +150,7 @@ def mlstm(h, mx, W, p, eps):
             S = keep * S + add * np.outer(k[t, hh], v[t, hh])
             n = keep * n + add * k[t, hh]
             m = m2
-            out[t, hh] = S.T @ q[t, hh] / (max(abs(n @ q[t, hh]), np.exp(-m)) + 1e-6)
+            out[t, hh] = S.T @ q[t, hh] / divisor(n @ q[t, hh], m)
     y = rms_unit(out, eps).reshape(T, H * V) * W[p + "norm"]
     return (y * sigmoid(h @ W[p + "g"].T)) @ W[p + "o"].T
 
