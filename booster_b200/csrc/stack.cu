@@ -184,6 +184,8 @@ struct StackModel {
     int max_slots = 0, max_eff = 0, max_exp = 0;      // routed mixtures: choices per token, expert width, experts
     size_t max_scan_state = 0;            // outer-product recurrences: the largest matrix state of a layer
     int max_scan_dim = 0, max_scan_heads = 0;
+    size_t max_sel_state = 0;             // selective scan: the largest inner x state; the most channels
+    int max_sel_inner = 0;
     float residual_mult = 1.f, embed_scale = 1.f;     // BLOCK_POSTNORM: factor on a sub-layer's normed output; on the embedding row
     bool unit_qk = false;                 // the design's attention has unit queries and keys
     const char * pair_default[2] = { "sigmoid_attention", "retention" };      // mixers of a pair whose branches name none
@@ -238,6 +240,7 @@ struct StackCtx {
     std::vector<float *> cache_allocs;    // the caches with their zero margins (caches[] point behind the front margin)
     float * att_part = nullptr, * att_ml = nullptr;   // key-slice partials of the latent attention (decode)
     float * scan_sb = nullptr, * scan_ac = nullptr;      // outer-product recurrences, long portions: per-chunk states [heads][chunks][state], decays [heads][chunks]
+    float * sel_l = nullptr, * sel_sum = nullptr;        // selective scan, long portions: what the segments leave
     float * den = nullptr;                // mLSTM: n . q [cap][heads]
     float * keep = nullptr;               // depth average: [layers + 1][cap][E] results of this pass's tokens
     float * Xp = nullptr, * Ap = nullptr, * Yk = nullptr, * r_wt = nullptr, * r_sg = nullptr;      // routed mixture: rows by slot, weights, shared gate
@@ -249,6 +252,7 @@ struct StackCtx {
     int sm_count = 148;
     __nv_bfloat16 * xb = nullptr;         // activations of a prompt pass rounded to bfloat16 (operand of the tcgen05 product)
     size_t xb_elems = 0;
+    float * xpart = nullptr;              // sums of the K parts of a product with few output tiles
     int * d_err = nullptr, * h_err = nullptr;   // raised by a kernel whose bounded wait ran out
     bool taps = false;
     std::vector<float> tap_data;
@@ -638,6 +642,7 @@ void load_selscan(StackModel & m, LayerSpec & L, const Json & mx, const safetens
     L.o = up_mat(m, sf.read_f32(p + "o", {E, n}), E, n, nullptr);
     m.weight_bytes += (int64_t) n * (N + taps + 2) * 4;
     L.n_rec = (size_t) n * N + (size_t) (taps - 1) * n;
+    m.max_sel_state = std::max(m.max_sel_state, (size_t) n * N); m.max_sel_inner = std::max(m.max_sel_inner, n);
     m.maxP = std::max(m.maxP, 2 * n); m.maxA = std::max(m.maxA, n); m.maxCV = std::max(m.maxCV, n);
     m.maxBG = std::max(m.maxBG, (R + 2 * N + 3) / 4 * 4);
 }
@@ -1136,9 +1141,15 @@ bool umma_enabled() {
     static const bool on = [] { const char * e = std::getenv("BOOSTER_B200_STACK_UMMA"); return !(e && e[0] == '0'); }();
     return on;
 }
+bool split_k_enabled() {
+    static const bool on = [] { const char * e = std::getenv("BOOSTER_B200_STACK_SPLIT_K"); return !(e && e[0] == '0'); }();
+    return on;
+}
+constexpr int GEMV_FEW_ROWS = 512;
 // what the tcgen05 product needs beside its operands: room for the activations rounded to bfloat16 and the error flag its
 // bounded waits raise
-struct UmmaScratch { __nv_bfloat16 * xb = nullptr; size_t elems = 0; int * err = nullptr; };
+struct UmmaScratch { __nv_bfloat16 * xb = nullptr; size_t elems = 0; int * err = nullptr; float * part = nullptr; int sm_count = 148; };
+size_t umma_part_floats(int sm_count) { return (size_t) sm_count * UM_BM * UM_BN; }      // one K part of an output tile per SM
 
 // what a product may ask for beyond its operands: the gated unit's kind and constants (y = g sigmoid(alpha g) (u + shift), g and u clamped
 // at +-limit, or gelu(g) u), rows sorted into segments per batch entry (tile kernels), an indexed batch (mat-vec)
@@ -1168,7 +1179,10 @@ void linear_on(cudaStream_t st, int dtype, int64_t * launches, const float * X, 
             if (dtype == STACK_F32) k_gemv<float, 2><<<grid, 256, 0, st>>>(a); else k_gemv<__nv_bfloat16, 2><<<grid, 256, 0, st>>>(a);
         } else {
             const dim3 grid((unsigned) ((N + 7) / 8), 1, (unsigned) batch);
-            if (dtype == STACK_F32) k_gemv<float, 1><<<grid, 256, 0, st>>>(a); else k_gemv<__nv_bfloat16, 1><<<grid, 256, 0, st>>>(a);
+            if (batch == 1 && N <= GEMV_FEW_ROWS && K >= 1024) {       // few, long rows: a block each
+                if (dtype == STACK_F32) k_gemv<float, 1, 8><<<(unsigned) N, 256, 0, st>>>(a); else k_gemv<__nv_bfloat16, 1, 8><<<(unsigned) N, 256, 0, st>>>(a);
+            }
+            else if (dtype == STACK_F32) k_gemv<float, 1><<<grid, 256, 0, st>>>(a); else k_gemv<__nv_bfloat16, 1><<<grid, 256, 0, st>>>(a);
         }
     } else if (dtype == STACK_BF16 && a.vec && us && us->xb && umma_enabled() && T >= 64 && N >= 128 && K >= 64 && (size_t) xbatch * T * K <= us->elems) {
         // tensor memory path: activations to bfloat16 once, then tcgen05.mma over cp.async-fed stages
@@ -1176,7 +1190,14 @@ void linear_on(cudaStream_t st, int dtype, int64_t * launches, const float * X, 
         if (!attr) throw std::runtime_error("cannot reserve shared memory for k_gemm_bf16_umma");
         k_to_bf16<<<dim3((unsigned) std::min((K + 255) / 256, 64), (unsigned) T, (unsigned) xbatch), 256, 0, st>>>(X, ldx, T, K, sX, us->xb, (long long) T * K);
         const dim3 grid((unsigned) ((N + UM_BN - 1) / UM_BN), (unsigned) ((T + UM_BM - 1) / UM_BM), (unsigned) batch);
-        k_gemm_bf16_umma<<<grid, 256, UM_SMEM, st>>>(a, us->xb, (long long) T * K, us->err);
+        const int tiles = (int) (grid.x * grid.y), nk = (K + UM_BK - 1) / UM_BK;
+        const int ksplit = batch == 1 && !a.glu && !a.seg && us->part && split_k_enabled() ? std::min(us->sm_count / tiles, nk / 4) : 1;
+        if (ksplit > 1) {
+            k_gemm_bf16_umma<<<dim3(grid.x, grid.y, (unsigned) ksplit), 256, UM_SMEM, st>>>(a, us->xb, (long long) T * K, us->err, ksplit, us->part);
+            k_split_sum<<<dim3((unsigned) ((N + 255) / 256), (unsigned) T), 256, 0, st>>>(us->part, ksplit, T, N, bias, Y, ldy);
+            if (launches) (*launches)++;
+        }
+        else k_gemm_bf16_umma<<<grid, 256, UM_SMEM, st>>>(a, us->xb, (long long) T * K, us->err);
         if (launches) (*launches)++;
     } else if (dtype == STACK_BF16 && a.vec && mma_enabled()) {
         const dim3 grid((unsigned) ((N + MM_BN - 1) / MM_BN), (unsigned) ((T + MM_BM - 1) / MM_BM), (unsigned) batch);
@@ -1190,7 +1211,7 @@ void linear_on(cudaStream_t st, int dtype, int64_t * launches, const float * X, 
 
 void linear(StackCtx * c, const float * X, int ldx, const DMat & W, float * Y, int ldy, int T, int batch = 1, long long sX = 0, long long sY = 0, bool glu = false, float glu_limit = 0.f,
             const LinOpt * opt = nullptr) {
-    const UmmaScratch us{c->xb, c->xb_elems, c->d_err};
+    const UmmaScratch us{c->xb, c->xb_elems, c->d_err, c->xpart, c->sm_count};
     linear_on(c->st, c->m->dtype, &c->launches, X, ldx, W.w, W.bias, Y, ldy, T, W.N, W.K, batch, sX, (long long) W.N * W.K, sY, glu, glu_limit, &us, opt);
 }
 
@@ -1538,13 +1559,13 @@ void mixer_mlstm(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
     if (T == 1) {
         OuterToken t{};
         t.P = c->P; t.q_off = 0; t.k_off = HD; t.v_off = 2 * HD; t.g_off = 2 * HD + HV; t.i_off = gi; t.f_off = gi + H;
-        t.q_scale = q_scale; t.cap = L.gate_cap; t.w = L.dnorm; t.m_state = m_state; t.m_stride = 1;
+        t.q_scale = q_scale; t.cap = L.gate_cap; t.w = L.dnorm; t.m_state = m_state;
         t.H = H; t.D = D; t.V = V; t.eps = c->m->eps; t.S = S; t.head_stride = (long long) L.head_stride; t.A = c->A;
         launch_outer_token<TOKEN_MLSTM>(c, t);
         linear(c, c->A, HV, L.o, c->out, E, T);
         return;
     }
-    k_mlstm_gates<<<H, 32, 0, c->st>>>(c->P, ldp, gi, gi + H, L.gate_cap, T, H, m_state, 1, c->BG, ldg);
+    k_mlstm_gates<<<H, 256, (size_t) 3 * T * 4, c->st>>>(c->P, ldp, gi, gi + H, L.gate_cap, T, H, m_state, c->BG, ldg);
     OuterScan s{};
     s.Q = c->P; s.K = c->P + HD; s.Vv = c->P + 2 * HD; s.ldq = s.ldk = s.ldv = ldp;
     s.T = T; s.H = H; s.share = 1; s.D = D; s.V = V; s.kind = SCAN_TABLE; s.ab = c->BG; s.ld_ab = ldg; s.S = S; s.head_stride = (long long) L.head_stride;
@@ -1578,10 +1599,17 @@ void mixer_ssd(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
     linear(c, c->A, inner, L.o, c->out, E, T);
 }
 
+constexpr int SEL_SEG = 64;               // tokens per segment of a long portion
 template <int LANES, int NS>
 void launch_selective(StackCtx * c, const LayerSpec & L, const SelScan & s) {
     const int nblk = (s.inner + 256 / LANES - 1) / (256 / LANES);
-    if (s.T > 1) k_selective_scan<LANES, NS><<<nblk, 256, 0, c->st>>>(s);
+    if (s.T >= SCAN_CHUNK_MIN_T && s.L && scan_chunks_enabled()) {
+        const unsigned rest = (unsigned) ((s.T + s.seg - 1) / s.seg - 1);
+        k_selective_scan<LANES, NS, SEL_FIRST><<<dim3((unsigned) nblk, rest), 256, 0, c->st>>>(s);
+        k_selective_scan<LANES, NS, SEL_REST><<<dim3((unsigned) nblk, rest), 256, 0, c->st>>>(s);
+        c->launches++;
+    }
+    else if (s.T > 1) k_selective_scan<LANES, NS, SEL_WHOLE><<<nblk, 256, 0, c->st>>>(s);
     else if (c->m->dtype == STACK_F32) k_selective_token<float, LANES, NS><<<nblk, 256, (size_t) L.dt_rank * 4, c->st>>>(s, (const float *) L.wdt.w, L.wdt.bias, L.dt_rank);
     else k_selective_token<__nv_bfloat16, LANES, NS><<<nblk, 256, (size_t) L.dt_rank * 4, c->st>>>(s, (const __nv_bfloat16 *) L.wdt.w, L.wdt.bias, L.dt_rank);
     c->launches++;
@@ -1594,7 +1622,7 @@ void mixer_selscan(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) 
     causal_conv(c, ConvArgs{c->P, 2 * n, 0, L.wconv, 0, hist, 0, c->CV, n, 0, T, n, L.taps, 1, 0, nullptr, nullptr, 0, 0, 0, L.bconv});
     linear(c, c->CV, n, L.wx, c->BG, ldb, T);
     if (T > 1) linear(c, c->BG, ldb, L.wdt, c->O, n, T);
-    const SelScan s{c->CV, n, c->O, n, c->BG, ldb, L.dt_rank, L.dt_rank + N, c->P + n, 2 * n, L.A_log, L.skip, S, T, n, N, c->A};
+    const SelScan s{c->CV, n, c->O, n, c->BG, ldb, L.dt_rank, L.dt_rank + N, c->P + n, 2 * n, L.A_log, L.skip, S, T, n, N, c->A, SEL_SEG, c->sel_l, c->sel_sum};
     if (N <= 16) launch_selective<4, 4>(c, L, s);
     else if (N <= 32) launch_selective<8, 4>(c, L, s);
     else if (N <= 64) launch_selective<16, 4>(c, L, s);
@@ -2146,13 +2174,13 @@ void stack_ctx_free(StackCtx * c) {
     cudaFree(c->d_out_tokens); cudaFree(c->d_counter);
     for (float * p : c->pools) cudaFree(p);
     for (float * p : { c->XS, c->VF }) cudaFree(p);
-    for (float * p : { c->Y2, c->U, c->XC, c->keep, c->scan_sb, c->scan_ac, c->den, c->Xp, c->Ap, c->Yk, c->r_wt, c->r_sg, c->r_z }) cudaFree(p);
+    for (float * p : { c->Y2, c->U, c->XC, c->keep, c->scan_sb, c->scan_ac, c->sel_l, c->sel_sum, c->den, c->Xp, c->Ap, c->Yk, c->r_wt, c->r_sg, c->r_z }) cudaFree(p);
     cudaFree(c->r_counter);
     for (int32_t * p : { c->r_sel, c->r_slot, c->r_src, c->r_seg }) cudaFree(p);
     for (float * p : { c->X, c->Hn, c->Y, c->P, c->A, c->QK, c->OL, c->CV, c->BG, c->O, c->rec, c->d_logits }) cudaFree(p);
     for (float * p : c->cache_allocs) cudaFree(p);
     cudaFree(c->att_scores); cudaFree(c->da_part); cudaFree(c->da_counter);
-    cudaFree(c->xb); cudaFree(c->d_err); cudaFreeHost(c->h_err);
+    cudaFree(c->xb); cudaFree(c->xpart); cudaFree(c->d_err); cudaFreeHost(c->h_err);
     cudaFree(c->d_step); cudaFree(c->d_arg); cudaFree(c->att_part); cudaFree(c->att_ml);
     cudaFreeHost(c->h_step); cudaFreeHost(c->h_logits); cudaFreeHost(c->h_arg);
     if (c->ev0) { cudaEventDestroy(c->ev0); cudaEventDestroy(c->ev1); }
@@ -2167,6 +2195,9 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
     SCU(cudaSetDevice(m->device));
     try {
         SCU(cudaStreamCreateWithFlags(&c->st, cudaStreamNonBlocking));
+        cudaDeviceProp prop;
+        SCU(cudaGetDeviceProperties(&prop, m->device));
+        c->sm_count = prop.multiProcessorCount;
         const size_t cap = (size_t) c->cap;
         // zero-filled: rows that a tile computes beyond the portion, and cached rows no token has written, must hold finite numbers
         const auto fl = [&](float ** p, size_t n) { SCU(cudaMalloc(p, std::max<size_t>(n, 4) * 4)); SCU(cudaMemsetAsync(*p, 0, std::max<size_t>(n, 4) * 4, c->st)); };
@@ -2179,6 +2210,10 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
         if (m->block == BLOCK_HYPER) fl(&c->XS, (size_t) m->streams * cap * m->E);
         if (m->vfirst_width > 0) fl(&c->VF, cap * (size_t) m->vfirst_width);
         if (m->max_scan_heads > 0) fl(&c->den, cap * (size_t) m->max_scan_heads);
+        if (m->max_sel_state > 0 && c->cap >= SCAN_CHUNK_MIN_T) {
+            const size_t nseg = (size_t) (c->cap + SEL_SEG - 1) / SEL_SEG;
+            fl(&c->sel_l, nseg * m->max_sel_state); fl(&c->sel_sum, nseg * (size_t) m->max_sel_inner);
+        }
         if (m->max_scan_state > 0 && c->cap >= SCAN_CHUNK_MIN_T) {
             const size_t nch = (size_t) (c->cap + RC - 1) / RC;
             fl(&c->scan_sb, nch * m->max_scan_state); fl(&c->scan_ac, nch * (size_t) m->max_scan_heads);
@@ -2203,14 +2238,12 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
         if (m->dtype == STACK_BF16) {
             c->xb_elems = std::max(cap * (size_t) std::max({ 2 * m->E, m->maxA, m->maxOL, m->maxP }), moe_rows * (size_t) std::max(m->E, m->max_eff));
             SCU(cudaMalloc(&c->xb, c->xb_elems * 2));
+            SCU(cudaMalloc(&c->xpart, umma_part_floats(c->sm_count) * 4));
         }
         SCU(cudaMalloc(&c->d_err, 4)); SCU(cudaMemsetAsync(c->d_err, 0, 4, c->st));
         SCU(cudaMallocHost(&c->h_err, 4)); *c->h_err = 0;
         c->caches.assign((size_t) m->n_caches, nullptr);
         c->pools.assign((size_t) m->n_caches, nullptr);
-        cudaDeviceProp prop;
-        SCU(cudaGetDeviceProperties(&prop, m->device));
-        c->sm_count = prop.multiProcessorCount;
         size_t smem = 0, part = 0, ml = 0, da_part = 0, da_cnt = 0;
         struct Cached { const LayerSpec * L; int index; };
         std::vector<Cached> cached;           // every attention cache of every run (a pair's branches each have their own)
@@ -2475,7 +2508,7 @@ float stack_time_linear(int device, int dtype, int T, int N, int K, int reps) {
         SCU(cudaMalloc(&X, (size_t) T * K * 4)); SCU(cudaMalloc(&Y, (size_t) T * N * 4)); SCU(cudaMalloc(&W, wbytes * copies));
         SCU(cudaMemset(X, 0, (size_t) T * K * 4)); SCU(cudaMemset(W, 0, wbytes * copies));
         us.elems = (size_t) T * K;
-        SCU(cudaMalloc(&us.xb, us.elems * 2)); SCU(cudaMalloc(&us.err, 4)); SCU(cudaMemset(us.err, 0, 4));
+        SCU(cudaMalloc(&us.xb, us.elems * 2)); SCU(cudaMalloc(&us.part, umma_part_floats(us.sm_count) * 4)); SCU(cudaMalloc(&us.err, 4)); SCU(cudaMemset(us.err, 0, 4));
         SCU(cudaStreamCreate(&st)); SCU(cudaEventCreate(&e0)); SCU(cudaEventCreate(&e1));
         for (int i = 0; i < 3; i++) linear_on(st, dtype, nullptr, X, K, (char *) W + wbytes * (size_t) (i % copies), nullptr, Y, N, T, N, K, 1, 0, 0, 0, false, 0.f, &us);
         SCU(cudaStreamSynchronize(st));
@@ -2485,11 +2518,11 @@ float stack_time_linear(int device, int dtype, int T, int N, int K, int reps) {
         SCU(cudaStreamSynchronize(st));
         cudaEventElapsedTime(&ms, e0, e1);
     } catch (...) {
-        cudaFree(X); cudaFree(Y); cudaFree(W); cudaFree(us.xb); cudaFree(us.err);
+        cudaFree(X); cudaFree(Y); cudaFree(W); cudaFree(us.xb); cudaFree(us.part); cudaFree(us.err);
         if (st) cudaStreamDestroy(st);
         throw;
     }
-    cudaFree(X); cudaFree(Y); cudaFree(W); cudaFree(us.xb); cudaFree(us.err);
+    cudaFree(X); cudaFree(Y); cudaFree(W); cudaFree(us.xb); cudaFree(us.part); cudaFree(us.err);
     cudaEventDestroy(e0); cudaEventDestroy(e1); cudaStreamDestroy(st);
     return ms / (float) std::max(reps, 1);
 }
@@ -2510,17 +2543,17 @@ void stack_linear(int device, int dtype, int T, int N, int K, const float * x, c
         SCU(cudaMalloc(&X, (size_t) T * K * 4)); SCU(cudaMalloc(&Y, (size_t) T * ny * 4));
         SCU(cudaMemcpy(X, x, (size_t) T * K * 4, cudaMemcpyHostToDevice));
         us.elems = (size_t) T * K;
-        SCU(cudaMalloc(&us.xb, us.elems * 2)); SCU(cudaMalloc(&us.err, 4)); SCU(cudaMemset(us.err, 0, 4));
+        SCU(cudaMalloc(&us.xb, us.elems * 2)); SCU(cudaMalloc(&us.part, umma_part_floats(us.sm_count) * 4)); SCU(cudaMalloc(&us.err, 4)); SCU(cudaMemset(us.err, 0, 4));
         linear_on(nullptr, dtype, nullptr, X, K, d.w, d.bias, Y, ny, T, N, K, 1, 0, 0, 0, glu != 0, limit, &us);
         SCU(cudaDeviceSynchronize());
         SCU(cudaMemcpy(y, Y, (size_t) T * ny * 4, cudaMemcpyDeviceToHost));
         SCU(cudaMemcpy(&herr, us.err, 4, cudaMemcpyDeviceToHost));
     } catch (...) {
-        cudaFree(X); cudaFree(Y); cudaFree(us.xb); cudaFree(us.err);
+        cudaFree(X); cudaFree(Y); cudaFree(us.xb); cudaFree(us.part); cudaFree(us.err);
         for (void * p : tmp.allocs) cudaFree(p);
         throw;
     }
-    cudaFree(X); cudaFree(Y); cudaFree(us.xb); cudaFree(us.err);
+    cudaFree(X); cudaFree(Y); cudaFree(us.xb); cudaFree(us.part); cudaFree(us.err);
     for (void * p : tmp.allocs) cudaFree(p);
     if (herr) throw std::runtime_error("k_gemm_bf16_umma gave up waiting for its pipeline");
 }

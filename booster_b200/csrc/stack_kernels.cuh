@@ -185,11 +185,13 @@ __device__ __forceinline__ float gated_unit(const LinArgs & a, float gate, float
 }
 
 constexpr int GEMV_MAX_T = 4;
-// decode and very short portions: one warp per output row, the row of W streamed once with 16-byte loads
-template <typename WT, int RPW>
+// decode and very short portions: one warp per output row, the row of W streamed once with 16-byte loads. WPR = 8 (matrices with too
+// few rows to fill the SMs): the block's 8 warps share one row and add their sums in a fixed order
+template <typename WT, int RPW, int WPR = 1>
 __global__ void __launch_bounds__(256) k_gemv(const LinArgs a) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int n = (blockIdx.x * (blockDim.x >> 5) + warp) * RPW;      // RPW = 2: a (gate, up) pair per warp
+    const int n = (WPR > 1 ? (int) blockIdx.x : blockIdx.x * (blockDim.x >> 5) + warp) * RPW;      // RPW = 2: a (gate, up) pair per warp
+    const int part = WPR > 1 ? warp : 0;
     if (n >= a.N) return;
     const int wi = a.w_index ? a.w_index[blockIdx.z] : (int) blockIdx.z;
     if (a.n_w > 0 && wi >= a.n_w) return;
@@ -204,7 +206,7 @@ __global__ void __launch_bounds__(256) k_gemv(const LinArgs a) {
     if (a.vec) {
         // U chunks of 16 bytes per row and lane are requested before any is used: a mat-vec is bound by the bytes in flight
         constexpr int U = RPW == 2 ? 2 : 4;
-        for (int kb = lane * VEC; kb < a.K; kb += 32 * VEC * U) {
+        for (int kb = (part * U * 32 + lane) * VEC; kb < a.K; kb += 32 * VEC * U * WPR) {
             uint4 raw[RPW][U];
 #pragma unroll
             for (int u = 0; u < U; u++) {
@@ -246,7 +248,7 @@ __global__ void __launch_bounds__(256) k_gemv(const LinArgs a) {
             }
         }
     } else {
-        for (int k = lane; k < a.K; k += 32) {
+        for (int k = part * 32 + lane; k < a.K; k += 32 * WPR) {
 #pragma unroll
             for (int r = 0; r < RPW; r++) {
                 const float wv = wf(w, (size_t) r * a.K + k);
@@ -254,6 +256,19 @@ __global__ void __launch_bounds__(256) k_gemv(const LinArgs a) {
                 for (int t = 0; t < GEMV_MAX_T; t++) if (t < a.T) acc[r][t] = fmaf(wv, x[(size_t) t * a.ldx + k], acc[r][t]);
             }
         }
+    }
+    if constexpr (WPR > 1) {
+        __shared__ float sums[RPW][GEMV_MAX_T][WPR];
+#pragma unroll
+        for (int r = 0; r < RPW; r++)
+#pragma unroll
+            for (int t = 0; t < GEMV_MAX_T; t++) if (t < a.T) { const float v = warp_sum(acc[r][t]); if (lane == 0) sums[r][t][warp] = v; }
+        __syncthreads();
+        if (warp != 0) return;
+#pragma unroll
+        for (int r = 0; r < RPW; r++)
+#pragma unroll
+            for (int t = 0; t < GEMV_MAX_T; t++) if (t < a.T) acc[r][t] = lane < WPR ? sums[r][t][lane] : 0.f;
     }
 #pragma unroll
     for (int t = 0; t < GEMV_MAX_T; t++) {
@@ -553,6 +568,8 @@ __global__ void __launch_bounds__(256) k_gemm_bf16_mma(const LinArgs a) {
 //              K = 64 deep; the activations were rounded to bfloat16 by k_to_bf16 beforehand
 //   issue      one thread: four K = 16 MMAs per stage, tcgen05.commit -> the stage's mbarrier (frees the stage for the refill)
 //   epilogue   warp w owns TMEM lanes 32 (w & 3) .. + 31 (= tokens) and column half w >> 2: tcgen05.ld, bias / gated unit, stores
+// Products with too few output tiles to fill the SMs are cut along K (ksplit > 1: blockIdx.z is the part): every part leaves its sums
+// in part [ksplit][T][N] and k_split_sum adds them in order, with the bias.
 // Every wait on an mbarrier is bounded: on a timeout the CTA raises *err, skips what is left and still frees its tensor memory.
 __global__ void k_to_bf16(const float * __restrict__ X, int ldx, int T, int K, long long sX, __nv_bfloat16 * __restrict__ Xb, long long sXb) {
     const float * x = X + (size_t) blockIdx.z * sX + (size_t) blockIdx.y * ldx;
@@ -577,7 +594,7 @@ __device__ __forceinline__ bool mbar_wait_limited(uint32_t bar, uint32_t parity,
     atomicExch(err, 1);
     return false;
 }
-__global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, const __nv_bfloat16 * __restrict__ Xb, long long sXb, int * err) {
+__global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, const __nv_bfloat16 * __restrict__ Xb, long long sXb, int * err, int ksplit = 1, float * __restrict__ part = nullptr) {
     extern __shared__ uint8_t um_raw[];
     __shared__ __align__(8) uint64_t done[UM_STAGES];
     __shared__ uint32_t tmem_base_s;
@@ -587,8 +604,9 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
     const int m0 = blockIdx.y * UM_BM, n0 = blockIdx.x * UM_BN;
     const int r0 = a.seg ? a.seg[blockIdx.z] : 0, T = a.seg ? a.seg[blockIdx.z + 1] - r0 : a.T;
     if (m0 >= T) return;                      // the whole block, before anything is allocated
-    const __nv_bfloat16 * X = a.seg ? Xb + (size_t) r0 * a.K : Xb + (size_t) blockIdx.z * sXb;
-    const __nv_bfloat16 * W = reinterpret_cast<const __nv_bfloat16 *>(a.W) + (size_t) blockIdx.z * a.sW;
+    const int bz = ksplit > 1 ? 0 : blockIdx.z;
+    const __nv_bfloat16 * X = a.seg ? Xb + (size_t) r0 * a.K : Xb + (size_t) bz * sXb;
+    const __nv_bfloat16 * W = reinterpret_cast<const __nv_bfloat16 *>(a.W) + (size_t) bz * a.sW;
     volatile int * failed = &failed_s;
     if (tid == 0) {
         failed_s = 0;
@@ -603,11 +621,12 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = tmem_base_s;
-    const int nk = (a.K + UM_BK - 1) / UM_BK;
+    const int nk_all = (a.K + UM_BK - 1) / UM_BK, kbeg = ksplit > 1 ? (int) ((long long) nk_all * blockIdx.z / ksplit) : 0;
+    const int nk = (ksplit > 1 ? (int) ((long long) nk_all * (blockIdx.z + 1) / ksplit) : nk_all) - kbeg;       // at least one: ksplit <= nk_all
     // one stage: 128 x 8 chunks of A (4 per thread) and 256 x 8 chunks of B (8 per thread); a warp's 32 chunks are 512 contiguous bytes
     const auto issue_copies = [&](int kt, int slot) {
         const uint32_t sa = smem0 + (uint32_t) slot * UM_STAGE_BYTES, sb = sa + UM_A_BYTES;
-        const int k0 = kt * UM_BK;
+        const int k0 = (kbeg + kt) * UM_BK;
 #pragma unroll
         for (int i = 0; i < 12; i++) {
             const int idx = tid + 256 * (i < 4 ? i : i - 4);
@@ -665,7 +684,9 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
     if (ok) {
         const int m = m0 + 32 * (warp & 3) + lane, cbase = (warp >> 2) * (UM_BN / 2);
         const uint32_t taddr = tmem + ((uint32_t) (32 * (warp & 3)) << 16) + (uint32_t) cbase;
-        float * Y = (a.seg ? a.Y + (size_t) r0 * a.ldy : a.Y + (size_t) blockIdx.z * a.sY) + (size_t) m * a.ldy;
+        const int ldy = ksplit > 1 ? a.N : a.ldy;
+        const float * bias = ksplit > 1 ? nullptr : a.bias;
+        float * Y = (ksplit > 1 ? part + (size_t) blockIdx.z * T * a.N : a.seg ? a.Y + (size_t) r0 * ldy : a.Y + (size_t) blockIdx.z * a.sY) + (size_t) m * ldy;
 #pragma unroll 1
         for (int c = 0; c < UM_BN / 2; c += 16) {
             float v[16];
@@ -678,11 +699,11 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (m < T) {
                 const int nb = n0 + cbase + c;
-                if (!a.glu && nb + 15 < a.N && (a.ldy & 3) == 0 && ((uintptr_t) (Y + nb) & 15) == 0) {       // whole 16-byte stores
+                if (!a.glu && nb + 15 < a.N && (ldy & 3) == 0 && ((uintptr_t) (Y + nb) & 15) == 0) {       // whole 16-byte stores
 #pragma unroll
                     for (int j = 0; j < 16; j += 4) {
                         float4 o = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
-                        if (a.bias) { o.x += a.bias[nb + j]; o.y += a.bias[nb + j + 1]; o.z += a.bias[nb + j + 2]; o.w += a.bias[nb + j + 3]; }
+                        if (bias) { o.x += bias[nb + j]; o.y += bias[nb + j + 1]; o.z += bias[nb + j + 2]; o.w += bias[nb + j + 3]; }
                         *reinterpret_cast<float4 *>(Y + nb + j) = o;
                     }
                     continue;
@@ -691,10 +712,10 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
                 for (int j = 0; j < 16; j += 2) {
                     const int n = n0 + cbase + c + j;
                     if (a.glu) {
-                        if (n + 1 < a.N) Y[n >> 1] = gated_unit(a, v[j] + (a.bias ? a.bias[n] : 0.f), v[j + 1] + (a.bias ? a.bias[n + 1] : 0.f));
+                        if (n + 1 < a.N) Y[n >> 1] = gated_unit(a, v[j] + (bias ? bias[n] : 0.f), v[j + 1] + (bias ? bias[n + 1] : 0.f));
                     } else {
-                        if (n < a.N) Y[n] = v[j] + (a.bias ? a.bias[n] : 0.f);
-                        if (n + 1 < a.N) Y[n + 1] = v[j + 1] + (a.bias ? a.bias[n + 1] : 0.f);
+                        if (n < a.N) Y[n] = v[j] + (bias ? bias[n] : 0.f);
+                        if (n + 1 < a.N) Y[n + 1] = v[j + 1] + (bias ? bias[n + 1] : 0.f);
                     }
                 }
             }
@@ -706,6 +727,22 @@ __global__ void __launch_bounds__(256, 1) k_gemm_bf16_umma(const LinArgs a, cons
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" :: "r"(tmem), "r"(256u) : "memory");
     }
+}
+
+// Y[t][n] = bias[n] + the parts' sums, in order
+__global__ void k_split_sum(const float * __restrict__ part, int ksplit, int T, int N, const float * __restrict__ bias, float * __restrict__ Y, int ldy) {
+    const int t = blockIdx.y, n = blockIdx.x * blockDim.x + threadIdx.x;
+    if (n >= N) return;
+    const float * p = part + (size_t) t * N + n;
+    const size_t plane = (size_t) T * N;
+    float v = bias ? bias[n] : 0.f;
+    int z = 0;
+    for (; z + 4 <= ksplit; z += 4) {
+        const float p0 = p[(size_t) z * plane], p1 = p[(size_t) (z + 1) * plane], p2 = p[(size_t) (z + 2) * plane], p3 = p[(size_t) (z + 3) * plane];
+        v = (((v + p0) + p1) + p2) + p3;
+    }
+    for (; z < ksplit; z++) v += p[(size_t) z * plane];
+    Y[(size_t) t * ldy + n] = v;
 }
 
 // ---- minGRU: S_t = (1 - z) S_(t-1) + z * cand, gates from the current token only ----------------------------------------

@@ -376,36 +376,41 @@ __device__ __forceinline__ float mlstm_log_in(float raw, float cap) { return cap
 __device__ __forceinline__ float mlstm_log_keep(float raw, float cap) { return log_sigmoidf_(cap * tanhf(raw / cap)); }
 // the read-out's divisor, from n . q (scaled like the query) and m
 __device__ __forceinline__ float mlstm_divisor(float nq, float m) { return fmaxf(fabsf(nq), expf(-m)) + 1e-6f; }
-// portions of several tokens: AB[t] = [ a: H | b: H | m: H ]. One warp per head; lanes hold 32 tokens' log gates, the maximum itself
-// is carried from token to token in order (two dependent operations each). m_state [H] is part of the sequence's state.
-__global__ void __launch_bounds__(32) k_mlstm_gates(const float * __restrict__ P, int ldp, int i_off, int f_off, float cap, int T, int H,
-                                                    float * __restrict__ m_state, long long m_stride, float * __restrict__ AB, int ld_ab) {
-    const int h = blockIdx.x, lane = threadIdx.x;
-    float m = m_state[(size_t) h * m_stride];
-    float ri = 0.f, rf = 0.f;
-    if (lane < T) { ri = P[(size_t) lane * ldp + i_off + h]; rf = P[(size_t) lane * ldp + f_off + h]; }
-    for (int t0 = 0; t0 < T; t0 += 32) {
-        const int t = t0 + lane, nt = min(32, T - t0);
-        const float li = mlstm_log_in(ri, cap), lf = mlstm_log_keep(rf, cap);
-        if (t + 32 < T) { ri = P[(size_t) (t + 32) * ldp + i_off + h]; rf = P[(size_t) (t + 32) * ldp + f_off + h]; }
-        float before = m, mine = m;
-#pragma unroll
-        for (int k = 0; k < 32; k++) {
-            const float fk = __shfl_sync(0xffffffffu, lf, k), ik = __shfl_sync(0xffffffffu, li, k);
-            if (k < nt) {
-                const float mk = fmaxf(fk + m, ik);
-                if (k == lane) { before = m; mine = mk; }
-                m = mk;
-            }
-        }
-        if (t < T) {
-            float * o = AB + (size_t) t * ld_ab;
-            o[h] = expf(lf + before - mine);
-            o[H + h] = expf(li - mine);
-            o[2 * H + h] = mine;
-        }
+// portions of several tokens: AB[t] = [ a: H | b: H | m: H ]. One block per head: log gates of all tokens at once into shared memory
+// (3 T floats, dynamic), the maximum from token to token in order by one warp (two dependent operations each), then a and b of
+// all tokens at once. m_state [H] is part of the sequence's state.
+__global__ void __launch_bounds__(256) k_mlstm_gates(const float * __restrict__ P, int ldp, int i_off, int f_off, float cap, int T, int H,
+                                                     float * __restrict__ m_state, float * __restrict__ AB, int ld_ab) {
+    extern __shared__ float msm[];
+    float * li = msm, * lf = msm + T, * mx = msm + 2 * T;
+    const int h = blockIdx.x;
+    const float m0 = m_state[h];
+    for (int t = threadIdx.x; t < T; t += blockDim.x) {
+        li[t] = mlstm_log_in(P[(size_t) t * ldp + i_off + h], cap);
+        lf[t] = mlstm_log_keep(P[(size_t) t * ldp + f_off + h], cap);
     }
-    if (lane == 0) m_state[(size_t) h * m_stride] = m;
+    __syncthreads();
+    if (threadIdx.x < 32) {
+        float m = m0;
+        int t = 0;
+        for (; t + 8 <= T; t += 8) {
+            float f[8], i[8];
+#pragma unroll
+            for (int k = 0; k < 8; k++) { f[k] = lf[t + k]; i[k] = li[t + k]; }
+#pragma unroll
+            for (int k = 0; k < 8; k++) { m = fmaxf(f[k] + m, i[k]); if (threadIdx.x == 0) mx[t + k] = m; }
+        }
+        for (; t < T; t++) { m = fmaxf(lf[t] + m, li[t]); if (threadIdx.x == 0) mx[t] = m; }
+        if (threadIdx.x == 0) m_state[h] = m;
+    }
+    __syncthreads();
+    for (int t = threadIdx.x; t < T; t += blockDim.x) {
+        float * o = AB + (size_t) t * ld_ab;
+        const float m = mx[t];
+        o[h] = expf(lf[t] + (t ? mx[t - 1] : m0) - m);
+        o[H + h] = expf(li[t] - m);
+        o[2 * H + h] = m;
+    }
 }
 
 // ---- one token, a whole mixer core in one launch: gates, state update, read-out, its norm and gate; one block per head -----------
@@ -423,7 +428,7 @@ struct OuterToken {
     float cap; const float * w;
     int H, D, V; float eps;
     float * S; long long head_stride;           // [D][V], then n [D] (mLSTM)
-    float * m_state; long long m_stride;
+    float * m_state;
     float * A;
 };
 template <int DMAX, int KIND>
@@ -436,10 +441,17 @@ __global__ void __launch_bounds__(512) k_outer_token(const OuterToken a) {
     const float * q = a.P + a.q_off + (size_t) h * D, * k = a.P + a.k_off + (size_t) h * D;
     float g, b = 1.f, m = 0.f;
     if constexpr (KIND == TOKEN_MLSTM) {
-        const float li = mlstm_log_in(a.P[a.i_off + h], a.cap), lf = mlstm_log_keep(a.P[a.f_off + h], a.cap), m0 = a.m_state[(size_t) h * a.m_stride];
+        const float li = mlstm_log_in(a.P[a.i_off + h], a.cap), lf = mlstm_log_keep(a.P[a.f_off + h], a.cap), m0 = a.m_state[h];
         m = fmaxf(lf + m0, li);
         g = expf(lf + m0 - m); b = expf(li - m);
     } else g = a.decay[h];
+    float * Sh = a.S + (size_t) h * a.head_stride;
+    constexpr int NL = (DMAX + 31) / 32;                // mLSTM: warp 0 keeps the normaliser, a lane every 32nd entry
+    float nv[NL];
+    if (KIND == TOKEN_MLSTM && warp == 0) {
+#pragma unroll
+        for (int i = 0; i < NL; i++) nv[i] = lane + 32 * i < D ? Sh[(size_t) D * V + lane + 32 * i] : 0.f;
+    }
     for (int i = tid; i < 2 * DMAX; i += blockDim.x) {
         const bool is_k = i >= DMAX;
         const int d = is_k ? i - DMAX : i, at = (d / DR) * (DR + GD_PAD) + d % DR;
@@ -457,35 +469,47 @@ __global__ void __launch_bounds__(512) k_outer_token(const OuterToken a) {
         (is_k ? ks : qs)[at] = v;
     }
     __syncthreads();
-    if (KIND == TOKEN_MLSTM && tid == 0) a.m_state[(size_t) h * a.m_stride] = m;       // every thread has read the old one
-    float * Sh = a.S + (size_t) h * a.head_stride;
-    const int base = rg * (DR + GD_PAD), cl = warp * 8 + (lane >> 2), cols = V + (KIND == TOKEN_MLSTM ? 1 : 0);
+    if (KIND == TOKEN_MLSTM && warp == 0) {
+        if (lane == 0) a.m_state[h] = m;                // every thread has read the old one
+        float nq = 0.f;
+#pragma unroll
+        for (int i = 0; i < NL; i++) {
+            const int d = lane + 32 * i, at = (d / DR) * (DR + GD_PAD) + d % DR;
+            if (d < D) {
+                nv[i] = fmaf(g, nv[i], ks[at] * b);
+                Sh[(size_t) D * V + d] = nv[i];
+                nq = fmaf(nv[i], qs[at], nq);
+            }
+        }
+        nq = warp_sum(nq);
+        if (lane == 0) o_s[V] = nq;
+    }
+    const int base = rg * (DR + GD_PAD), cl = warp * 8 + (lane >> 2);
     float ss = 0.f;
-    for (int c0 = 0; c0 < cols; c0 += ncols) {
+    for (int c0 = 0; c0 < V; c0 += ncols) {
         const int col = c0 + cl;
-        const bool live = col < cols, is_n = KIND == TOKEN_MLSTM && col == V;
-        const float v = live ? (is_n ? b : b * a.P[a.v_off + (size_t) h * V + col]) : 0.f;
-        const size_t rstep = is_n ? 1 : V;
-        float * Sc = Sh + (is_n ? (size_t) D * V : (size_t) col);
+        const bool live = col < V;
+        const float v = live ? b * a.P[a.v_off + (size_t) h * V + col] : 0.f;
+        float * Sc = Sh + col;
         float op[4] = { 0.f, 0.f, 0.f, 0.f };
         constexpr int CH = DR < 16 ? DR : 16;           // rows whose loads are in flight together (the stores would order them otherwise)
 #pragma unroll 1
         for (int i0 = 0; i0 < DR; i0 += CH) {
             float sv[CH];
 #pragma unroll
-            for (int i = 0; i < CH; i++) { const int d = rg * DR + i0 + i; sv[i] = (live && d < D) ? Sc[(size_t) d * rstep] : 0.f; }
+            for (int i = 0; i < CH; i++) { const int d = rg * DR + i0 + i; sv[i] = (live && d < D) ? Sc[(size_t) d * V] : 0.f; }
 #pragma unroll
             for (int i = 0; i < CH; i++) {
                 const int d = rg * DR + i0 + i;
                 sv[i] = fmaf(g, sv[i], ks[base + i0 + i] * v);
-                if (live && d < D) Sc[(size_t) d * rstep] = sv[i];
+                if (live && d < D) Sc[(size_t) d * V] = sv[i];
                 op[i & 3] = fmaf(sv[i], qs[base + i0 + i], op[i & 3]);
             }
         }
         float o = (op[0] + op[1]) + (op[2] + op[3]);
         o += __shfl_xor_sync(0xffffffffu, o, 1);
         o += __shfl_xor_sync(0xffffffffu, o, 2);
-        if (rg == 0 && live) { o_s[col] = o; if (!is_n) ss = fmaf(o, o, ss); }
+        if (rg == 0 && live) { o_s[col] = o; ss = fmaf(o, o, ss); }
     }
     ss = warp_sum(ss);
     if (lane == 0) red[warp] = ss;
@@ -557,6 +581,14 @@ __global__ void __launch_bounds__(1024) k_gated_part_norm(const float * __restri
 // whole portion: LANES neighbouring lanes share a channel, each holding NS of its entries. The inputs of TT tokens arrive in shared
 // memory by asynchronous copies while the tokens before them are walked (two buffers); step sizes and gates are taken there once per
 // (token, channel).
+// Long portions are cut into segments of `seg` tokens that run side by side. A segment takes the state before it to
+// exp(A sum_t dt_t) S + L, with L what it leaves when it starts from zero, so:
+//   SEL_FIRST   segments 0 .. n - 2: segment 0 is the walk itself from the sequence's state, the others start from zero and write
+//               nothing but L; all leave L (segment 0: the state after it) and their sum of step sizes
+//   SEL_REST    segments 1 .. n - 1: the entry state folded from what the segments before left, then the walk; the last one
+//               leaves the sequence's state
+// SEL_WHOLE is the walk over a short portion.
+enum { SEL_WHOLE = 0, SEL_FIRST = 1, SEL_REST = 2 };
 struct SelScan {
     const float * X; int ldx;               // convolved inputs [T][inner]
     const float * dt; int ldt;              // raw step sizes (bias included) [T][inner]
@@ -566,32 +598,37 @@ struct SelScan {
     float * S;
     int T, inner, N;
     float * A;                              // [T][inner]
+    int seg;                                // tokens per segment
+    float * L; float * sum;                 // [segments][inner][N], [segments][inner]
 };
-template <int LANES, int NS>
+template <int LANES, int NS, int MODE>
 __global__ void __launch_bounds__(256) k_selective_scan(const SelScan a) {
     constexpr int NCH = 256 / LANES, NM = LANES * NS, TT = NM > 64 ? 8 : 16;
     __shared__ __align__(16) float xs[2][TT][NCH], ds[2][TT][NCH], zs[2][TT][NCH], bs[2][TT][NM], cs[2][TT][NM];
     const int tid = threadIdx.x, rg = tid % LANES, cl = tid / LANES, c0 = blockIdx.x * NCH, c = c0 + cl, N = a.N;
     const bool live = c < a.inner;
+    const int sg = MODE == SEL_WHOLE ? 0 : MODE == SEL_FIRST ? blockIdx.y : blockIdx.y + 1;
+    const int T0 = MODE == SEL_WHOLE ? 0 : sg * a.seg, T1 = MODE == SEL_WHOLE ? a.T : min(a.T, T0 + a.seg);
+    const bool emits = MODE != SEL_FIRST || sg == 0;
     const auto stage = [&](int t0, int buf) {
-        const int nt = min(TT, a.T - t0);
+        const int nt = min(TT, T1 - t0);
         for (int i = tid; i < nt * NCH; i += 256) {
             const int tt = i / NCH, k = i % NCH;
             const bool in = c0 + k < a.inner;
             const size_t t = (size_t) (t0 + tt), ch = in ? c0 + k : 0;
             cp_async4(&xs[buf][tt][k], a.X + t * a.ldx + ch, in);
             cp_async4(&ds[buf][tt][k], a.dt + t * a.ldt + ch, in);
-            cp_async4(&zs[buf][tt][k], a.Z + t * a.ldz + ch, in);
+            if (emits) cp_async4(&zs[buf][tt][k], a.Z + t * a.ldz + ch, in);
         }
         for (int i = tid; i < nt * NM; i += 256) {
             const int tt = i / NM, n = i % NM;
             const bool in = n < N;
             const float * p = a.BC + (size_t) (t0 + tt) * a.ldb + (in ? n : 0);
             cp_async4(&bs[buf][tt][n], p + a.b_off, in);
-            cp_async4(&cs[buf][tt][n], p + a.c_off, in);
+            if (emits) cp_async4(&cs[buf][tt][n], p + a.c_off, in);
         }
     };
-    stage(0, 0);
+    stage(T0, 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
     float s[NS], rate[NS];
     float * Sc = a.S + (size_t) (live ? c : 0) * N;
@@ -599,25 +636,47 @@ __global__ void __launch_bounds__(256) k_selective_scan(const SelScan a) {
     for (int i = 0; i < NS; i++) {
         const int n = rg * NS + i;
         const bool in = live && n < N;
-        s[i] = in ? Sc[n] : 0.f;
+        s[i] = in && (MODE == SEL_WHOLE || (MODE == SEL_FIRST && sg == 0)) ? Sc[n] : 0.f;
         rate[i] = in ? -1.4426950408889634f * expf(a.A_log[(size_t) c * N + n]) : 0.f;      // in powers of two
     }
+    if (MODE == SEL_REST) {
+        for (int k = 0; k < sg; k++) {
+            const size_t at = (size_t) k * a.inner + (live ? c : 0);
+            const float sum = a.sum[at];
+#pragma unroll
+            for (int i = 0; i < NS; i++) { const int n = rg * NS + i; if (live && n < N) s[i] = fmaf(exp2f(sum * rate[i]), s[i], a.L[at * N + n]); }
+        }
+    }
     const float skip = live ? a.skip[c] : 0.f;
-    for (int t0 = 0, buf = 0; t0 < a.T; t0 += TT, buf ^= 1) {
-        const int nt = min(TT, a.T - t0);
-        if (t0 + TT < a.T) stage(t0 + TT, buf ^ 1);
+    float total = 0.f;
+    for (int t0 = T0, buf = 0; t0 < T1; t0 += TT, buf ^= 1) {
+        const int nt = min(TT, T1 - t0);
+        if (t0 + TT < T1) stage(t0 + TT, buf ^ 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
         for (int i = tid; i < nt * NCH; i += 256) {
             float & d = ds[buf][i / NCH][i % NCH], & z = zs[buf][i / NCH][i % NCH];
-            d = softplusf_(d); z = siluf_(z);
+            d = softplusf_(d);
+            if (emits) z = siluf_(z);
         }
         __syncthreads();
+        if (!emits) {
+#pragma unroll 4
+            for (int tt = 0; tt < nt; tt++) {
+                const float dt = ds[buf][tt][cl], dx = dt * xs[buf][tt][cl];
+                total += dt;
+#pragma unroll
+                for (int i = 0; i < NS; i++) s[i] = fmaf(exp2f(dt * rate[i]), s[i], dx * bs[buf][tt][rg * NS + i]);
+            }
+            __syncthreads();
+            continue;
+        }
 #pragma unroll 4
         for (int tt = 0; tt < nt; tt++) {
             const float dt = ds[buf][tt][cl], x = xs[buf][tt][cl], dx = dt * x;
             float y = 0.f;
+            if (MODE == SEL_FIRST) total += dt;
 #pragma unroll
             for (int i = 0; i < NS; i++) {
                 s[i] = fmaf(exp2f(dt * rate[i]), s[i], dx * bs[buf][tt][rg * NS + i]);
@@ -629,9 +688,12 @@ __global__ void __launch_bounds__(256) k_selective_scan(const SelScan a) {
         }
         __syncthreads();
     }
+    if (MODE == SEL_REST && T1 < a.T) return;           // only the last segment's state is the sequence's
     if (live) {
+        float * to = MODE == SEL_FIRST ? a.L + ((size_t) sg * a.inner + c) * N : Sc;
 #pragma unroll
-        for (int i = 0; i < NS; i++) { const int n = rg * NS + i; if (n < N) Sc[n] = s[i]; }
+        for (int i = 0; i < NS; i++) { const int n = rg * NS + i; if (n < N) to[n] = s[i]; }
+        if (MODE == SEL_FIRST && rg == 0) a.sum[(size_t) sg * a.inner + c] = total;
     }
 }
 // one token: the step size's low-rank product (Wdt [inner][R], bias) is part of the same launch; the lanes of a channel share it

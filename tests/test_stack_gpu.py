@@ -397,6 +397,10 @@ def test_bad_models_fail_loudly(tmp_path):
     ("bfloat16", 200, 300, 136, False), ("bfloat16", 130, 512, 64, True),     # tcgen05 + TMEM: ragged and whole tiles
     ("bfloat16", 513, 258, 1032, False),                                      # more K steps than pipeline stages, several token tiles
     ("bfloat16", 70, 130, 35, False),                                         # odd K: CUDA cores
+    ("bfloat16", 512, 168, 2048, False), ("bfloat16", 100, 131, 584, False),  # few output tiles: K in parts, rows of whole and of ragged 16-byte chunks
+    ("bfloat16", 200, 600, 4104, False),
+    ("bfloat16", 1, 37, 2048, False), ("bfloat16", 3, 160, 4096, False), ("float32", 2, 20, 1028, False),      # few long rows: eight warps each
+    ("float32", 4, 11, 1031, False),
     ("float32", 50, 70, 33, True), ("float32", 3, 9, 7, False)], ids=str)
 def test_products_pick_their_kernel_and_agree_with_numpy(dtype, T, N, K, glu):
     rng = np.random.default_rng(T * 1000 + N)
