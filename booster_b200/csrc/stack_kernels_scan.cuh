@@ -154,7 +154,7 @@ __device__ __forceinline__ void async_copies_done() {
 // grid (H, chunks, ceil(V / NC)), 256 threads: thread (ty, tx) owns 8 x NC / 16 of a 128 x NC tile of U_c; keys and values of the
 // chunk are staged in shared memory
 template <int NC>
-__global__ void __launch_bounds__(256) k_outer_chunk_kv(const OuterScan a, int vec, float * __restrict__ SB, float * __restrict__ AC) {
+__global__ void __launch_bounds__(256, NC == 128 ? 2 : 1) k_outer_chunk_kv(const OuterScan a, int vec, float * __restrict__ SB, float * __restrict__ AC) {
     constexpr int CW = NC / 16;
     __shared__ __align__(16) float Ks[RC][128], Vs[RC][NC];
     __shared__ float pw[RC];
