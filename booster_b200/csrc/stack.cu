@@ -1,10 +1,10 @@
 // stack.cu — the layer-stack model family on the B200 engine: configuration (config.json), weights (model.safetensors),
 // per-sequence state (attention cache + recurrent state), the step function for prompt portions and single tokens, and
 // the registry of designs and mixers. Kernels: stack_kernels.cuh, stack_kernels_mix.cuh,
-// stack_kernels_hyper.cuh, stack_kernels_scan.cuh. C-ABI dispatch: engine.cu.
+// stack_kernels_hyper.cuh, stack_kernels_scan.cuh, stack_kernels_side.cuh. C-ABI dispatch: engine.cu.
 //
 // A design is a name in config.json ("architecture") mapped to a builder that turns the configuration into a list of
-// LayerSpec; a mixer is a name ("type") mapped to a loader of its tensors and a forward routine. Five designs are registered:
+// LayerSpec; a mixer is a name ("type") mapped to a loader of its tensors and a forward routine. Six designs are registered:
 //   Matulorn   sequential sub-layers with grouped norms before and after each; mixers minGRU | latent attention (rotated
 //              part, window, sink) | gated delta rule; clamped gated feed-forward
 //   Dopilorn   both sub-layers read the same residual (x += mixer(n1 x) + ff(n2 x)) behind a causal convolution of their
@@ -27,6 +27,11 @@
 //              window beside a selective scan, each normed, averaged) | mLSTM | state-space duality (mamba2). Feed-forward: gelu
 //              unit | routed mixture (soft-max over experts and identity outputs, a correction on the choice, normalised
 //              weights, clamped units, a gated shared unit)
+//   Bozisun    embedding plus a row hashed from each pair of neighbouring tokens; both sub-layers read one normed input
+//              (x += mixer(n x) + ff(n x)), then the layer adds an input of the token's own (a slice of a per-token table, gated by x,
+//              projected and normed). Mixer: soft-max attention over grouped heads (every earlier position, normed queries and keys,
+//              YaRN rotation, gated entry by entry). Feed-forward: silu unit | routed mixture (biased logits, soft-max over the
+//              chosen); a span of layers run several times; soft-capped logits
 // A model is executed as a list of layer RUNS: (layer, state slot), one per layer unless the design repeats some.
 #include "stack.hpp"
 #include "safetensors.hpp"
@@ -34,6 +39,7 @@
 #include "stack_kernels_mix.cuh"
 #include "stack_kernels_hyper.cuh"
 #include "stack_kernels_scan.cuh"
+#include "stack_kernels_side.cuh"
 
 #include <algorithm>
 #include <cmath>
@@ -52,7 +58,7 @@ using namespace stk;
 namespace {
 
 enum MixerKind { MIX_MINGRU = 0, MIX_LATENT, MIX_DELTA, MIX_GDELTA, MIX_DIFFATTN, MIX_RETENTION, MIX_SIGATTN, MIX_PAIR, MIX_GQATTN, MIX_SELSCAN, MIX_MLSTM, MIX_SSD };
-enum BlockKind { BLOCK_SEQUENTIAL = 0, BLOCK_PARALLEL, BLOCK_PRENORM, BLOCK_HYPER, BLOCK_POSTNORM };
+enum BlockKind { BLOCK_SEQUENTIAL = 0, BLOCK_PARALLEL, BLOCK_PRENORM, BLOCK_HYPER, BLOCK_POSTNORM, BLOCK_SHARED };
 enum FfKind { FF_GLU = 0, FF_POLY, FF_MOE };
 constexpr int CHUNK_MAX = 512;          // tokens per pass of a prompt portion (longer steps run as several passes)
 constexpr float GLU_ALPHA = 1.702f;     // the feed-forward's sigmoid slope: fixed by the design
@@ -107,7 +113,8 @@ struct LayerSpec {
     float * corr = nullptr;              // added to the scores when experts are chosen, not when they are weighed
     bool norm_w = false;                 // the chosen scores are divided by their sum
     float r_scale = 1.f;
-    int route_fn = 0;                    // 0: soft-max over the experts; 1: sigmoid of each logit
+    int route_fn = 0;                    // 0: soft-max over the experts; 1: sigmoid of each logit; 2: soft-max over the chosen logits
+    float * r_bias = nullptr;            // added to the router's logits
     bool scale_input = false;            // the choice's weight multiplies the expert's input instead of its output
     float * router = nullptr, * w_sg = nullptr;      // float32: the router is computed in 32-bit
     DMat e_gateup, e_down;
@@ -147,6 +154,11 @@ struct LayerSpec {
     // a pair of mixers side by side (MIX_PAIR): each over its root mean square times a weight, then their mean
     std::vector<LayerSpec> parts;
     float * pair_w[2] = { nullptr, nullptr };
+    // the token's own input, added at the end of the layer: x += norm(side_proj (gelu(side_gate x) e)) side_norm, e = entries side_off ..
+    // side_off + dim of the token's row of StackModel::side_table
+    DMat side_gate, side_proj;
+    float * side_norm = nullptr;
+    int side_off = 0;
     // parallel blocks: weights of the causal convolution in front of each sub-layer, [2][E][taps]
     float * canon = nullptr;
     // state a sequence keeps for one run of this layer
@@ -189,6 +201,11 @@ struct StackModel {
     float residual_mult = 1.f, embed_scale = 1.f;     // BLOCK_POSTNORM: factor on a sub-layer's normed output; on the embedding row
     bool unit_qk = false;                 // the design's attention has unit queries and keys
     const char * pair_default[2] = { "sigmoid_attention", "retention" };      // mixers of a pair whose branches name none
+    void * pair_table = nullptr;          // rows hashed from (previous token, token), added to the embedding: [buckets + 1][E], the last for a sequence's first token
+    int64_t pair_buckets = 0, pair_mul_prev = 0, pair_mul_cur = 0;
+    void * side_table = nullptr;          // inputs of the tokens' own: [vocab][layers x side_dim]
+    int side_dim = 0;
+    int max_dense = 0;                    // BLOCK_SHARED: widest dense feed-forward (its units have a buffer beside the mixer's)
     DMat loop_in;                         // repeated span: [E][2 E]
     float * loop_step = nullptr;          // [times][E]
     std::vector<LayerSpec> layers;
@@ -213,7 +230,11 @@ struct StepDev {                          // device image of a step's header
 struct StackCtx {
     StackModel * m = nullptr;
     int n_ctx = 0, n_past = 0, cap = 0;
+    int32_t last_token = -1;              // the sequence's newest token (-1: none yet)
     cudaStream_t st = nullptr;
+    cudaStream_t st2 = nullptr;           // BLOCK_SHARED, few-token steps: the feed-forward beside the mixer
+    cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
+    float * F = nullptr, * SZ = nullptr;  // BLOCK_SHARED: units of a dense feed-forward [cap][max_dense]; the token input's gate [cap][side_dim]
     float * XS = nullptr, * VF = nullptr; // hyper-connections: the streams [S][cap][E]; value mixing: the first mixing layer's values of this pass [cap][G V]
     std::vector<float *> pools;           // per attention cache: means of whole blocks of cached rows (nullptr: the layer keeps none)
     float * Y2 = nullptr, * U = nullptr, * XC = nullptr;     // parallel blocks: the feed-forward's output, the convolved inputs [2][cap][E], [x; x0] rows
@@ -321,6 +342,50 @@ void load_mingru(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
     m.maxP = std::max(m.maxP, 3 * w); m.maxA = std::max(m.maxA, w);
 }
 
+// rotary frequencies f_i = base^(-2i/dims) of a mixer's "rot" object (absent, or nothing to rotate: no rotation) on at most `most` entries.
+// "scaling" comes in two forms:
+//   {factor, fast, slow, original}   YaRN: i(t) = dims ln(original / (2 pi t)) / (2 ln base) is the pair that makes t turns over `original`
+//                                    positions; pairs from floor(i(fast)) to ceil(i(slow)) pass linearly from f to f / factor, and
+//                                    cos and sin grow by 0.1 ln(factor) + 1
+//   {factor, low, high, original}    a frequency of wavelength l = 2 pi / f stays when original / l > high, is divided by `factor` when
+//                                    original / l < low, and is blended linearly in original / l in between
+void load_rot(StackModel & m, LayerSpec & L, const Json & mx, int most) {
+    L.rope_dims = 0; L.rope_mag = 1.f;
+    std::vector<float> freq(1, 0.f);
+    if (most > 0 && mx.has("rot")) {
+        const Json & rot = mx.at("rot");
+        const int dims = L.rope_dims = (int) rot.integer("dims", most);
+        if (dims < 0 || dims > most || dims % 2) throw std::runtime_error("config: rot.dims must be even and at most the size of what is rotated (" + std::to_string(most) + ")");
+        const double base = rot.number("base");
+        freq.assign((size_t) std::max(dims / 2, 1), 0.f);
+        const bool scaled = rot.has("scaling"), yarn = scaled && rot.at("scaling").has("fast");
+        double factor = 1.0, low = 0, high = 0, orig = 0, lo = 0, hi = 0;
+        if (scaled) {
+            const Json & sc = rot.at("scaling");
+            factor = sc.number("factor"); orig = sc.number("original");
+            if (yarn) {
+                const auto pair_of = [&](double t) { return dims * std::log(orig / (2 * M_PI * t)) / (2 * std::log(base)); };
+                lo = std::max(std::floor(pair_of(sc.number("fast"))), 0.0);
+                hi = std::min(std::ceil(pair_of(sc.number("slow"))), (double) dims - 1);
+                L.rope_mag = (float) (0.1 * std::log(factor) + 1.0);
+            } else { low = sc.number("low"); high = sc.number("high"); }
+        }
+        for (int i = 0; i < dims / 2; i++) {
+            double f = std::pow(base, -2.0 * i / dims);
+            if (yarn) {
+                const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+                f = f / factor * ramp + f * (1.0 - ramp);
+            } else if (scaled) {
+                const double wave = 2.0 * M_PI / f;
+                if (wave > orig / low) f /= factor;
+                else if (!(wave < orig / high)) { const double s = (orig / wave - low) / (high - low); f = (1.0 - s) * f / factor + s * f; }
+            }
+            freq[(size_t) i] = (float) f;
+        }
+    }
+    L.rope_freq = up_f32(m, freq);
+}
+
 void load_latent(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) {
     const int E = m.E;
     const int H = L.H = need_int(mx, "heads"), D = L.D = need_int(mx, "dim"), R = L.R = (int) mx.integer("rot_dim", 0);
@@ -363,36 +428,7 @@ void load_latent(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
     L.uv = up_mat(m, sf.read_f32(p + "uv", {H * V, rank}), V, rank, nullptr, H);
     L.sink = sf.find(p + "sink") ? up_f32(m, sf.read_f32(p + "sink", {H})) : nullptr;
     L.o = up_mat(m, sf.read_f32(p + "o", {E, H * V}), E, H * V, nullptr);
-    // rotary frequencies: f_i = base^(-2i/dims), blended by YaRN when rot.scaling is given
-    L.rope_dims = 0; L.rope_mag = 1.f;
-    std::vector<float> freq(1, 0.f);
-    if (R > 0 && mx.has("rot")) {
-        const Json & rot = mx.at("rot");
-        const int dims = L.rope_dims = (int) rot.integer("dims", R);
-        if (dims < 0 || dims > R || dims % 2) throw std::runtime_error("config: rot.dims must be even and at most rot_dim");
-        const double base = rot.number("base");
-        freq.assign((size_t) std::max(dims / 2, 1), 0.f);
-        double factor = 1.0, lo = 0, hi = 0;
-        const bool yarn = rot.has("scaling");
-        if (yarn) {
-            const Json & sc = rot.at("scaling");
-            factor = sc.number("factor");
-            const double orig = sc.number("original"), fast = sc.number("fast"), slow = sc.number("slow");
-            const auto dim_of = [&](double t) { return dims * std::log(orig / (2 * M_PI * t)) / (2 * std::log(base)); };
-            lo = std::max(std::floor(dim_of(fast)), 0.0);
-            hi = std::min(std::ceil(dim_of(slow)), (double) dims - 1);
-            L.rope_mag = (float) (0.1 * std::log(factor) + 1.0);
-        }
-        for (int i = 0; i < dims / 2; i++) {
-            double f = std::pow(base, -2.0 * i / dims);
-            if (yarn) {
-                const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
-                f = f / factor * ramp + f * (1.0 - ramp);
-            }
-            freq[(size_t) i] = (float) f;
-        }
-    }
-    L.rope_freq = up_f32(m, freq);
+    load_rot(m, L, mx, R);
     L.cache_row = (size_t) rank + R;
     m.maxP = std::max(m.maxP, L.qdkv.N); m.maxA = std::max({ m.maxA, H * V, qr > 0 ? H * D : 0 });
     m.maxQK = std::max(m.maxQK, H * (rank + R)); m.maxOL = std::max(m.maxOL, H * rank);
@@ -489,34 +525,6 @@ void load_diffattn(StackModel & m, LayerSpec & L, const Json & mx, const safeten
     m.maxQK = std::max(m.maxQK, nq); m.maxOL = std::max(m.maxOL, H * V);      // prompt portions: regrouped queries, per-group outputs
 }
 
-// rotary frequencies f_i = base^(-2i/dims) of a mixer's "rot" object (absent: no rotation). With "scaling" {factor, low, high, original}
-// a frequency of wavelength l = 2 pi / f stays when original / l > high, is divided by `factor` when original / l < low, and is blended
-// linearly in original / l in between
-void load_rot(StackModel & m, LayerSpec & L, const Json & mx, int D) {
-    L.rope_dims = 0; L.rope_mag = 1.f;
-    std::vector<float> freq(1, 0.f);
-    if (mx.has("rot")) {
-        const Json & rot = mx.at("rot");
-        const int dims = L.rope_dims = (int) rot.integer("dims", D);
-        if (dims < 0 || dims > D || dims % 2) throw std::runtime_error("config: rot.dims must be even and at most dim");
-        const double base = rot.number("base");
-        freq.assign((size_t) std::max(dims / 2, 1), 0.f);
-        const bool scaled = rot.has("scaling");
-        double factor = 1.0, low = 0, high = 0, orig = 0;
-        if (scaled) { const Json & sc = rot.at("scaling"); factor = sc.number("factor"); low = sc.number("low"); high = sc.number("high"); orig = sc.number("original"); }
-        for (int i = 0; i < dims / 2; i++) {
-            double f = std::pow(base, -2.0 * i / dims);
-            if (scaled) {
-                const double wave = 2.0 * M_PI / f;
-                if (wave > orig / low) f /= factor;
-                else if (!(wave < orig / high)) { const double s = (orig / wave - low) / (high - low); f = (1.0 - s) * f / factor + s * f; }
-            }
-            freq[(size_t) i] = (float) f;
-        }
-    }
-    L.rope_freq = up_f32(m, freq);
-}
-
 // bookkeeping of a matrix state [heads][head_stride] walked by the outer-product recurrence
 void note_outer_state(StackModel & m, LayerSpec & L, int heads, int dim, size_t head_stride) {
     L.head_stride = head_stride;
@@ -577,8 +585,9 @@ void load_sigattn(StackModel & m, LayerSpec & L, const Json & mx, const safetens
 
 float read_scalar(const safetensors_file & sf, const std::string & name);
 // soft-max attention over grouped heads: '<prefix>{q,k,v,o}', optional 'q.norm' / 'k.norm' [dim], 'r1' / 'r2' [heads] (distance
-// penalty), 'sink' [heads], 'g' [heads][E] (output gate), 'vmix' (one number). Configuration: heads, kv_heads, dim, vdim, scale,
-// softcap, rot.{base,dims}, mask.{size,pool}, v_mix. The mask's kind belongs to the mixer's name (chunks | window).
+// penalty), 'sink' [heads], 'g' [heads][E] or [heads vdim][E] (output gate, one number per head or per entry), 'vmix' (one number).
+// Configuration: heads, kv_heads, dim, vdim, scale, softcap, rot.{base,dims,scaling}, mask.{size,pool}, v_mix. The mask's kind belongs
+// to the mixer's name (chunks | window | none: every earlier position).
 void load_gqattn(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p, int mask_kind) {
     const int E = m.E;
     const int H = L.H = need_int(mx, "heads"), G = L.KH = (int) mx.integer("kv_heads", H), D = L.D = need_int(mx, "dim"), V = L.V = need_int(mx, "vdim");
@@ -589,6 +598,7 @@ void load_gqattn(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
     if (L.cap < 0.f) throw std::runtime_error("config: softcap must not be negative");
     L.mask_kind = MASK_CAUSAL; L.window = 0; L.pool = 0;
     if (mx.has("mask")) {
+        if (mask_kind == MASK_CAUSAL) throw std::runtime_error("config: this attention sees every earlier position and takes no mask");
         L.mask_kind = mask_kind;
         L.window = need_int(mx.at("mask"), "size");
         if (mask_kind == MASK_WINDOW) L.pool = (int) mx.at("mask").integer("pool", 0);
@@ -600,7 +610,12 @@ void load_gqattn(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
     std::vector<float> W = sf.read_f32(p + "q", {H * D, E});
     append(W, sf.read_f32(p + "k", {G * D, E}));
     append(W, sf.read_f32(p + "v", {G * V, E}));
-    if (sf.find(p + "g")) { append(W, sf.read_f32(p + "g", {H, E})); L.head_gate = true; L.gate_rows = H; }
+    if (const st_tensor * gt = sf.find(p + "g")) {
+        if (gt->shape.size() != 2 || (gt->shape[0] != H && gt->shape[0] != (int64_t) H * V)) throw std::runtime_error("tensor '" + p + "g' must have heads or heads x vdim rows");
+        L.head_gate = true;
+        L.gate_rows = (int) gt->shape[0];
+        append(W, sf.read_f32(p + "g", {L.gate_rows, E}));
+    }
     L.proj = up_mat(m, W, H * D + G * D + G * V + L.gate_rows, E, nullptr);
     if (sf.find(p + "q.norm")) L.qw = up_f32(m, sf.read_f32(p + "q.norm", {D}));
     if (sf.find(p + "k.norm")) L.kw = up_f32(m, sf.read_f32(p + "k.norm", {D}));
@@ -622,6 +637,7 @@ void load_gqattn(StackModel & m, LayerSpec & L, const Json & mx, const safetenso
     m.maxQK = std::max(m.maxQK, H * D); m.maxOL = std::max(m.maxOL, H * V);
 }
 void load_gqattn_chunks(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) { load_gqattn(m, L, mx, sf, p, MASK_CHUNK); }
+void load_gqattn_causal(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) { load_gqattn(m, L, mx, sf, p, MASK_CAUSAL); }
 void load_gqattn_window(StackModel & m, LayerSpec & L, const Json & mx, const safetensors_file & sf, const std::string & p) { load_gqattn(m, L, mx, sf, p, MASK_WINDOW); }
 
 // selective scan: '<prefix>{in,conv,conv.b,x,dt,dt.b,A_log,D,o}'
@@ -708,6 +724,7 @@ const MixerEntry MIXERS[] = {
     { "parallel", MIX_PAIR, load_pair },
     { "chunk_attention", MIX_GQATTN, load_gqattn_chunks },
     { "window_attention", MIX_GQATTN, load_gqattn_window },
+    { "causal_attention", MIX_GQATTN, load_gqattn_causal },
     { "selective_scan", MIX_SELSCAN, load_selscan },
     { "mlstm", MIX_MLSTM, load_mlstm },
     { "mamba2", MIX_SSD, load_ssd },
@@ -755,6 +772,24 @@ void add_run(StackModel & m, int layer, int pass) {
     if (const int nc = n_layer_caches(L)) { r.cache_index = m.n_caches; m.n_caches += nc; }
     m.weight_bytes += L.bytes;
     m.runs.push_back(r);
+}
+
+// 'loop' of a configuration: layers start .. stop - 1 run `times` times in a row (absent: no such span)
+struct LoopSpan { int start = 0, stop = 0, times = 0; };
+LoopSpan read_loop(const Json & cfg, int n_layers) {
+    LoopSpan s;
+    if (!cfg.has("loop")) return s;
+    const Json & lp = cfg.at("loop");
+    s.start = need_int(lp, "start", 0); s.stop = need_int(lp, "stop", 0); s.times = need_int(lp, "times", 0);
+    if (s.start > s.stop || s.stop > n_layers) throw std::runtime_error("config: loop.start .. loop.stop must lie within the layers");
+    if (s.stop == s.start || s.times == 0) s = LoopSpan();
+    return s;
+}
+// the model's runs in order; with `opens`, the first run of every pass of the span carries the pass's number
+void add_runs(StackModel & m, int n_layers, const LoopSpan & s, bool opens) {
+    for (int i = 0; i < s.start; i++) add_run(m, i, -1);
+    for (int t = 0; t < s.times; t++) for (int i = s.start; i < s.stop; i++) add_run(m, i, opens && i == s.start ? t : -1);
+    for (int i = s.stop; i < n_layers; i++) add_run(m, i, -1);
 }
 
 // ---- designs ----------------------------------------------------------------------------------------------------------
@@ -873,20 +908,13 @@ void build_dopilorn(StackModel & m, const Json & cfg, const safetensors_file & s
         L.bytes = m.weight_bytes - bytes0;
         m.weight_bytes = bytes0;
     }
-    int start = 0, stop = 0, times = 0;
-    if (cfg.has("loop")) {
-        const Json & lp = cfg.at("loop");
-        start = need_int(lp, "start", 0); stop = need_int(lp, "stop", 0); times = need_int(lp, "times", 0);
-        if (start > stop || stop > n) throw std::runtime_error("config: loop.start .. loop.stop must lie within the layers");
-        if (stop > start && times > 0) {
-            m.loop_in = up_mat(m, sf.read_f32("loop.in", {E, 2 * E}), E, 2 * E, nullptr);
-            m.weight_bytes += m.loop_in.bytes * (times - 1);
-            m.loop_step = up_f32(m, sf.read_f32("loop.step", {times, E}));
-        } else { start = stop = times = 0; }
+    const LoopSpan span = read_loop(cfg, n);
+    if (span.times > 0) {
+        m.loop_in = up_mat(m, sf.read_f32("loop.in", {E, 2 * E}), E, 2 * E, nullptr);
+        m.weight_bytes += m.loop_in.bytes * (span.times - 1);
+        m.loop_step = up_f32(m, sf.read_f32("loop.step", {span.times, E}));
     }
-    for (int i = 0; i < start; i++) add_run(m, i, -1);
-    for (int t = 0; t < times; t++) for (int i = start; i < stop; i++) add_run(m, i, i == start ? t : -1);
-    for (int i = stop; i < n; i++) add_run(m, i, -1);
+    add_runs(m, n, span, true);
     m.final_norm = up_f32(m, one_plus(sf.read_f32("final.norm", {E})));
     m.head = up_mat(m, sf.read_f32("head", {m.vocab, E}), m.vocab, E, nullptr);
 }
@@ -911,8 +939,9 @@ DMat load_glu_pair(StackModel & m, const safetensors_file & sf, const std::strin
     return up_mat(m, W, 2 * ff, E, nullptr);
 }
 // what a design fixes about its routed mixture: the score function, where a choice's weight is applied, a gate on the shared unit;
-// scores chosen with a correction and normalised, identity outputs, and clamped units (slope GLU_ALPHA, shift 1, "limit") instead of silu ones
-struct MixtureKind { int route_fn; bool scale_input; bool shared_gate; bool corrected = false; bool clamped = false; };
+// scores chosen with a correction and normalised, identity outputs, clamped units (slope GLU_ALPHA, shift 1, "limit") instead of silu ones,
+// and a bias on the router's logits
+struct MixtureKind { int route_fn; bool scale_input; bool shared_gate; bool corrected = false; bool clamped = false; bool biased = false; };
 void load_mixture(StackModel & m, LayerSpec & L, const Json & mj, const safetensors_file & sf, const std::string & p, const MixtureKind & mk) {
     const int E = m.E;
     L.route_fn = mk.route_fn; L.scale_input = mk.scale_input;
@@ -931,6 +960,7 @@ void load_mixture(StackModel & m, LayerSpec & L, const Json & mj, const safetens
     const int ff = L.e_ff = need_int(mj.at("expert"), "ff");
     L.ff_kind = FF_MOE;
     L.router = up_f32(m, sf.read_f32(p + "router", {n, E}));
+    if (mk.biased) L.r_bias = up_f32(m, sf.read_f32(p + "router.b", {n}));
     if (mk.corrected) { L.corr = up_f32(m, sf.read_f32(p + "correction", {n})); L.norm_w = true; }
     if (mk.clamped) L.e_limit = (float) mj.at("expert").number("limit");
     else { L.act_alpha = 1.f; L.act_shift = 0.f; }
@@ -1122,6 +1152,79 @@ void build_kogerax(StackModel & m, const Json & cfg, const safetensors_file & sf
     m.head = up_mat(m, sf.read_f32("head", {m.vocab, E}), m.vocab, E, nullptr);
 }
 
+// Bozisun: x = embed[token] + pair[hash(previous token, token)] -> runs of layers (h = norm1(x); x += attention(h) + ff(h); x += the token's own
+// input of the layer) with a span of layers repeated -> norm -> head -> soft cap. Plain norm weights. The pair table, the token inputs,
+// the span, the cap and a layer's feed-forward may each be absent.
+void build_bozisun(StackModel & m, const Json & cfg, const safetensors_file & sf) {
+    m.block = BLOCK_SHARED;
+    m.vocab = need_int(cfg, "vocab"); m.E = need_int(cfg, "width");
+    m.eps = (float) cfg.at("norm").number("eps");
+    m.groups = 1;
+    m.softcap = (float) cfg.number("logit_softcap", 0.0);
+    const int E = m.E;
+    const auto table = [&](const std::string & name, int rows, int width) {       // rows are picked, not multiplied: no weight a token reads
+        DMat d = up_mat(m, sf.read_f32(name, {rows, width}), rows, width, nullptr);
+        m.weight_bytes -= d.bytes;
+        return d.w;
+    };
+    m.embed = table("embed", m.vocab, E);
+    const Json & layers = cfg.at("layers");
+    if (layers.kind != Json::Arr || layers.arr.empty()) throw std::runtime_error("config: 'layers' must be a non-empty list");
+    const int n = (int) layers.arr.size();
+    if (cfg.has("embedding") && cfg.at("embedding").has("bigram")) {
+        const Json & bj = cfg.at("embedding").at("bigram");
+        m.pair_buckets = need_int(bj, "buckets");
+        m.pair_mul_prev = need_int(bj, "mul_prev", 0); m.pair_mul_cur = need_int(bj, "mul_cur", 0);
+        m.pair_table = table("bigram", (int) m.pair_buckets + 1, E);
+    }
+    if (cfg.has("token_side")) {
+        m.side_dim = need_int(cfg.at("token_side"), "dim");
+        if ((int64_t) n * m.side_dim > (1 << 30)) throw std::runtime_error("config: token_side.dim is out of range");
+        m.side_table = table("side.embed", m.vocab, n * m.side_dim);
+    }
+    for (int i = 0; i < n; i++) {
+        const Json & lj = layers.arr[(size_t) i];
+        const std::string type = lj.string("type", ""), p = "l" + std::to_string(i) + ".";
+        if (type != "attention") throw std::runtime_error("config: layer " + std::to_string(i) + ": mixer '" + type + "' is not part of the Bozisun design");
+        const MixerEntry * me = &find_mixer("causal_attention", (size_t) i);
+        const int64_t bytes0 = m.weight_bytes;
+        m.layers.emplace_back();
+        LayerSpec & L = m.layers.back();
+        L.kind = me->kind;
+        L.has_mlp = lj.has("mlp");
+        L.norm1 = up_f32(m, sf.read_f32(p + "norm1", {E}));
+        me->load(m, L, lj.at("mixer"), sf, p + "mix.");
+        if (L.gate_rows != L.H * L.V) throw std::runtime_error("tensor '" + p + "mix.g' must have heads x vdim rows");
+        if (!L.qw || !L.kw) throw std::runtime_error("tensor '" + p + "mix.q.norm' or '" + p + "mix.k.norm' is missing");
+        if (L.has_mlp) {
+            const Json & mj = lj.at("mlp");
+            const std::string kind = mj.string("kind", "dense");
+            if (kind == "moe") {
+                if (mj.has("shared")) throw std::runtime_error("config: a shared unit is not part of the Bozisun design");
+                load_mixture(m, L, mj, sf, p + "mlp.", MixtureKind{2, false, false, false, false, true});
+            } else if (kind == "dense") {
+                L.ff = need_int(mj, "ff");
+                L.act_alpha = 1.f; L.act_shift = 0.f;          // g sigmoid(g) u
+                L.gateup = load_glu_pair(m, sf, p + "mlp.", L.ff, E, nullptr);
+                L.down = up_mat(m, sf.read_f32(p + "mlp.down", {E, L.ff}), E, L.ff, nullptr);
+                m.max_dense = std::max(m.max_dense, L.ff);
+            } else throw std::runtime_error("config: feed-forward kind '" + kind + "' is not part of the Bozisun design (dense | moe)");
+        }
+        if (m.side_dim > 0) {
+            L.side_gate = up_mat(m, sf.read_f32(p + "side.gate", {m.side_dim, E}), m.side_dim, E, nullptr);
+            L.side_proj = up_mat(m, sf.read_f32(p + "side.proj", {E, m.side_dim}), E, m.side_dim, nullptr);
+            L.side_norm = up_f32(m, sf.read_f32(p + "side.norm", {E}));
+            L.side_off = i * m.side_dim;
+        }
+        m.weight_bytes += (int64_t) E * 4 * (m.side_dim > 0 ? 2 : 1);
+        L.bytes = m.weight_bytes - bytes0;
+        m.weight_bytes = bytes0;
+    }
+    add_runs(m, n, read_loop(cfg, n), false);
+    m.final_norm = up_f32(m, sf.read_f32("final.norm", {E}));
+    m.head = up_mat(m, sf.read_f32("head", {m.vocab, E}), m.vocab, E, nullptr);
+}
+
 struct DesignEntry { const char * name; void (*build)(StackModel &, const Json &, const safetensors_file &); };
 const DesignEntry DESIGNS[] = {
     { "Matulorn", build_matulorn },
@@ -1129,6 +1232,7 @@ const DesignEntry DESIGNS[] = {
     { "Tosevik", build_tosevik },
     { "Rumurax", build_rumurax },
     { "Kogerax", build_kogerax },
+    { "Bozisun", build_bozisun },
 };
 
 // ---- launches ---------------------------------------------------------------------------------------------------------
@@ -1689,7 +1793,7 @@ bool gqa_tiles_enabled() {
     return on;
 }
 
-// soft-max attention over grouped heads: P[t] = [ q | k | v | head gates ] -> per-head norms, rotation, value mixing; keys and
+// soft-max attention over grouped heads: P[t] = [ q | k | v | output gates ] -> per-head norms, rotation, value mixing; keys and
 // values to the cache row of the token's position (and the means of the blocks this step completes to the pool) -> attention
 // under the layer's mask -> gate -> output product
 void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
@@ -1697,12 +1801,13 @@ void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
     float * cache = c->caches[(size_t) R.cache_index], * pool = c->pools[(size_t) R.cache_index];
     const StepState * st = &c->d_step->st;
     linear(c, c->in, E, L.proj, c->P, ldp, T);
-    const GqaPrepArgs pa{c->P, ldp, H, G, D, V, L.qw, L.kw, c->m->eps, RopeArgs{L.rope_freq, L.rope_dims, 1.0f, L.rope_adjacent ? 1 : 0}, st, c->CV, cache, row,
+    const GqaPrepArgs pa{c->P, ldp, H, G, D, V, L.qw, L.kw, c->m->eps, RopeArgs{L.rope_freq, L.rope_dims, L.rope_mag, L.rope_adjacent ? 1 : 0}, st, c->CV, cache, row,
                          c->VF, L.vmode, L.vlambda, L.unit_qk ? 1 : 0};
     k_gqa_prep<<<dim3((unsigned) T, T <= 16 ? (unsigned) ((H + G + 7) / 8) : 1u), 256, 0, c->st>>>(pa);      // few tokens: a token's heads over several blocks
     c->launches++;
     if (L.pool > 0) { k_pool_rows<<<dim3((unsigned) (T / L.pool + 1), (unsigned) ((row + 127) / 128)), 128, 0, c->st>>>(cache, row, pool, L.pool, st); c->launches++; }
     const float * gate = L.head_gate ? c->P + nq + row : nullptr;
+    const int gate_per_entry = L.head_gate && L.gate_rows == H * V && V > 1 ? 1 : 0;
     const GqaMask mask{L.mask_kind, L.window, L.pool};
     const GqaScore sc{L.scale, L.cap};
     if (T >= 8 && gqa_tiles_enabled()) {
@@ -1736,7 +1841,7 @@ void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
                               G, grp, V, (long long) Tpad * Rh * V, 1);
             c->launches++;
         }
-        k_group_o_layout<<<T, 256, 0, c->st>>>(c->OL, Tpad, H, G, V, c->A, gate, ldp);      // the head gates ride on the regrouping
+        k_group_o_layout<<<T, 256, 0, c->st>>>(c->OL, Tpad, H, G, V, c->A, gate, ldp, gate_per_entry);      // the gates ride on the regrouping
         c->launches += 2;
         linear(c, c->A, H * V, L.o, c->out, E, T);
         return;
@@ -1745,7 +1850,7 @@ void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
     const int blocks = ((T + TQ - 1) / TQ) * H;
     const int max_keys = L.mask_kind == MASK_CAUSAL ? c->n_ctx : std::min(c->n_ctx, L.window + (L.pool > 0 ? c->n_ctx / L.pool : 0));
     const int nsplit = std::max(1, std::min({ 2 * c->sm_count / blocks, ((max_keys + 31) / 32 + WPQ - 1) / WPQ, GQA_MAX_SPLIT }));
-    const GqaAttnArgs a{c->CV, nq, cache, pool, row, st, c->A, L.r1, L.r2, L.sink, gate, ldp, T, H, G, D, V, sc, mask, TQ,
+    const GqaAttnArgs a{c->CV, nq, cache, pool, row, st, c->A, L.r1, L.r2, L.sink, gate, ldp, gate_per_entry, T, H, G, D, V, sc, mask, TQ,
                         (D % 4 == 0 && row % 4 == 0 && ((uintptr_t) cache & 15) == 0 && ((uintptr_t) pool & 15) == 0) ? 1 : 0, nsplit, c->da_part, c->da_counter};
     const dim3 grid((unsigned) ((T + TQ - 1) / TQ), (unsigned) H, (unsigned) nsplit);
     const int VPL = gqa_vpl(L);
@@ -1886,7 +1991,7 @@ void enqueue_layers_parallel(StackCtx * c, int T) {
 // unit's in c->Y; the layer's join weighs and adds them
 void mixture_ff(StackCtx * c, const LayerSpec & L, const float * h, int T, const int32_t ** slot_of) {
     const int E = c->m->E, top = L.top, ff = L.e_ff, slots = T * top, n = L.n_exp + L.n_ident;
-    const RouteArgs ra{h, E, E, L.router, L.w_sg, n, top, L.n_groups, L.keep_groups, L.r_scale, c->r_sel, c->r_wt, c->r_sg, c->r_z, c->r_counter, L.route_fn, T <= 16 ? 8 : 1, L.corr, L.norm_w ? 1 : 0};
+    const RouteArgs ra{h, E, E, L.router, L.w_sg, n, top, L.n_groups, L.keep_groups, L.r_scale, c->r_sel, c->r_wt, c->r_sg, c->r_z, c->r_counter, L.route_fn, T <= 16 ? 8 : 1, L.corr, L.norm_w ? 1 : 0, L.r_bias};
     k_moe_route<<<dim3((unsigned) T, (unsigned) ((n + (L.w_sg ? 1 : 0) + 8 / ra.wpr - 1) / (8 / ra.wpr))), 256, (size_t) (2 * n + L.n_groups) * 4, c->st>>>(ra);
     c->launches++;
     LinOpt o;
@@ -2058,28 +2163,119 @@ void enqueue_layers_postnorm(StackCtx * c, int T) {
     SCU(cudaGetLastError());
 }
 
+bool fork_enabled() {
+    static const bool on = [] { const char * e = std::getenv("BOOSTER_B200_STACK_FORK"); return !(e && e[0] == '0'); }();
+    return on;
+}
+bool side_fused_enabled() {
+    static const bool on = [] { const char * e = std::getenv("BOOSTER_B200_STACK_SIDE_FUSED"); return !(e && e[0] == '0'); }();
+    return on;
+}
+// while it lives, launches go to the context's second stream
+struct SideStream {
+    StackCtx * c; bool on;
+    SideStream(StackCtx * c_, bool on_) : c(c_), on(on_) { if (on) std::swap(c->st, c->st2); }
+    ~SideStream() { if (on) std::swap(c->st, c->st2); }
+};
+
+// end of a layer of a shared-input block: X += Ya + Yb (or the mixture's choices), then the token's own input, then the norm nw -> Hn
+void layer_end(StackCtx * c, const LayerSpec & L, SumArgs a, const float * nw, int T) {
+    const StackModel & m = *c->m;
+    const int E = m.E, dim = m.side_dim, nt = hc_threads(T, E, 4);
+    a.X = c->X; a.E = E; a.eps = m.eps; a.Hn = c->Hn;
+    a.nw = dim > 0 ? nullptr : nw;
+    const SideW s{m.side_table, (int) m.layers.size() * dim, L.side_off, dim, L.side_gate.w, L.side_proj.w, L.side_norm};
+    const size_t smem = end_smem(E, dim);
+    if (dim > 0 && T <= GEMV_MAX_T && smem <= 40 * 1024 && side_fused_enabled()) {
+        const int vecw = m.dtype == STACK_F32 ? 4 : 8;
+        int lpr = 1;                                       // lanes per row of the projection: as many as it has 16-byte pieces
+        while (lpr < 32 && lpr * vecw < dim) lpr *= 2;
+        a.nw = nw;
+        const dim3 grid(END_CTAS, (unsigned) T);
+        const auto go = [&](auto kernel) { kernel<<<grid, END_THREADS, smem, c->st>>>(a, s, c->d_step->tokens, m.vocab, end_slice(E), E % vecw == 0 ? 1 : 0, dim % vecw == 0 ? 1 : 0, lpr); };
+        if (m.dtype == STACK_F32) go(k_layer_end<float>); else go(k_layer_end<__nv_bfloat16>);
+        c->launches++;
+        return;
+    }
+    if (E % 4 == 0) k_sum_join<4><<<T, nt, 0, c->st>>>(a);      // every buffer of a context is 16-byte aligned and its rows are E floats apart
+    else k_sum_join<1><<<T, hc_threads(T, E), 0, c->st>>>(a);
+    c->launches++;
+    if (dim <= 0) return;
+    linear(c, c->X, E, L.side_gate, c->SZ, dim, T);
+    const dim3 zgrid((unsigned) T, (unsigned) ((dim + 127) / 128));
+    if (m.dtype == STACK_F32) k_side_gate<float><<<zgrid, 128, 0, c->st>>>(c->SZ, s, c->d_step->tokens, m.vocab);
+    else k_side_gate<__nv_bfloat16><<<zgrid, 128, 0, c->st>>>(c->SZ, s, c->d_step->tokens, m.vocab);
+    linear(c, c->SZ, dim, L.side_proj, c->Y, E, T);
+    PostJoinArgs j{};
+    j.X = c->X; j.E = E; j.eps = m.eps; j.mult = 1.f; j.w = L.side_norm; j.scratch = c->Hn; j.Ya = c->Y; j.fw = nw; j.Hn = c->Hn;
+    if (E % 4 == 0) k_post_join<4><<<T, nt, 0, c->st>>>(j);
+    else k_post_join<1><<<T, hc_threads(T, E), 0, c->st>>>(j);
+    c->launches += 2;
+}
+
+// blocks whose two sub-layers read one normed input: h = norm1(x), x += mixer(h) + ff(h), then the token's own input. The norm of the
+// layer that follows (after the last one: the model's) is taken where a layer ends and left in c->Hn. Steps of few tokens run the
+// feed-forward beside the mixer on a second stream: neither fills the GPU, and nothing of one waits for the other.
+void enqueue_layers_shared(StackCtx * c, int T) {
+    StackModel & m = *c->m;
+    const int E = m.E, nt = hc_threads(T, E);
+    const float * w0 = m.layers[(size_t) m.runs[0].layer].norm1;
+    const PairTable pt{m.pair_table, (unsigned long long) m.pair_mul_prev, (unsigned long long) m.pair_mul_cur, (unsigned long long) m.pair_buckets};
+    if (m.dtype == STACK_F32) k_embed_pair<float><<<T, nt, 0, c->st>>>((const float *) m.embed, pt, &c->d_step->st, c->d_step->tokens, E, m.vocab, w0, m.eps, c->X, c->Hn);
+    else k_embed_pair<__nv_bfloat16><<<T, nt, 0, c->st>>>((const __nv_bfloat16 *) m.embed, pt, &c->d_step->st, c->d_step->tokens, E, m.vocab, w0, m.eps, c->X, c->Hn);
+    c->launches++;
+    for (size_t ri = 0; ri < m.runs.size(); ri++) {
+        const RunSpec & R = m.runs[ri];
+        const LayerSpec & L = m.layers[(size_t) R.layer];
+        const bool fork = L.has_mlp && T <= GEMV_MAX_T && fork_enabled();      // no product of such a step uses the tensor-core scratch, which is one per context
+        c->in = c->Hn; c->out = c->Y;
+        if (fork) { SCU(cudaEventRecord(c->ev_fork, c->st)); SCU(cudaStreamWaitEvent(c->st2, c->ev_fork, 0)); }
+        run_mixer(c, L, R, T);
+        SumArgs a{};
+        a.Ya = c->Y;
+        if (L.has_mlp) {
+            SideStream beside(c, fork);
+            if (L.ff_kind == FF_MOE) {
+                mixture_ff(c, L, c->Hn, T, &a.slot_of);
+                a.Yk = c->Yk; a.wt = c->r_wt; a.top = L.top;
+            } else {
+                LinOpt o;
+                o.glu_kind = L.act_kind; o.alpha = L.act_alpha; o.shift = L.act_shift;
+                linear(c, c->Hn, E, L.gateup, c->F, L.ff, T, 1, 0, 0, true, INFINITY, &o);
+                linear(c, c->F, L.ff, L.down, c->Y2, E, T);
+                a.Yb = c->Y2;
+            }
+            if (fork) SCU(cudaEventRecord(c->ev_join, c->st));
+        }
+        if (fork) SCU(cudaStreamWaitEvent(c->st, c->ev_join, 0));
+        layer_end(c, L, a, ri + 1 < m.runs.size() ? m.layers[(size_t) m.runs[ri + 1].layer].norm1 : m.final_norm, T);
+        if (c->taps) tap_layer(c, ri, T);
+    }
+    SCU(cudaGetLastError());
+}
+
 // the layers over the T tokens whose header (positions, ids) is already on the device
 void enqueue_layers(StackCtx * c, int T) {
     if (c->m->block == BLOCK_PARALLEL) enqueue_layers_parallel(c, T);
     else if (c->m->block == BLOCK_PRENORM) enqueue_layers_prenorm(c, T);
     else if (c->m->block == BLOCK_HYPER) enqueue_layers_hyper(c, T);
     else if (c->m->block == BLOCK_POSTNORM) enqueue_layers_postnorm(c, T);
+    else if (c->m->block == BLOCK_SHARED) enqueue_layers_shared(c, T);
     else enqueue_layers_sequential(c, T);
 }
 
 // final norm + head on n_rows rows of the pass (row indices in d_step->rows) -> d_logits[row_off ..]
 void enqueue_head(StackCtx * c, int n_rows, int64_t row_off, bool one_token = false) {
     StackModel & m = *c->m;
-    if (m.block == BLOCK_HYPER || m.block == BLOCK_POSTNORM) {
+    const bool normed = m.block == BLOCK_HYPER || m.block == BLOCK_POSTNORM || m.block == BLOCK_SHARED;
+    const float * hn = c->Hn;
+    if (normed) {
         // the last join left the normed residual (the sum of the streams) in Hn for every row of the pass: the wanted rows are gathered for the head
-        const float * hn = c->Hn;
         if (!one_token) { k_gather_rows<<<n_rows, 128, 0, c->st>>>(c->Hn, m.E, c->d_step->rows, m.E, c->Y); c->launches++; hn = c->Y; }
-        linear(c, hn, m.E, m.head, c->d_logits + row_off * m.vocab, m.vocab, n_rows);
-        return;
     }
-    if (m.dyt) { k_dyt_rows<<<n_rows, 256, 0, c->st>>>(c->X, m.E, c->d_step->rows, DytW{m.final_norm, m.final_b, m.final_alpha}, m.E, c->Hn, m.E); c->launches++; }
+    else if (m.dyt) { k_dyt_rows<<<n_rows, 256, 0, c->st>>>(c->X, m.E, c->d_step->rows, DytW{m.final_norm, m.final_b, m.final_alpha}, m.E, c->Hn, m.E); c->launches++; }
     else norm(c, c->X, m.E, c->d_step->rows, m.final_norm, m.E, m.groups, c->Hn, m.E, n_rows, false);
-    linear(c, c->Hn, m.E, m.head, c->d_logits + row_off * m.vocab, m.vocab, n_rows);
+    linear(c, hn, m.E, m.head, c->d_logits + row_off * m.vocab, m.vocab, n_rows);
     if (m.softcap > 0.f) {
         const size_t n = (size_t) n_rows * m.vocab;
         k_softcap<<<(unsigned) ((n + 255) / 256), 256, 0, c->st>>>(c->d_logits + row_off * m.vocab, n, m.softcap);
@@ -2172,6 +2368,10 @@ void stack_ctx_free(StackCtx * c) {
     if (c->g_token) cudaGraphExecDestroy(c->g_token);
     if (c->g_greedy) cudaGraphExecDestroy(c->g_greedy);
     cudaFree(c->d_out_tokens); cudaFree(c->d_counter);
+    cudaFree(c->F); cudaFree(c->SZ);
+    if (c->ev_fork) cudaEventDestroy(c->ev_fork);
+    if (c->ev_join) cudaEventDestroy(c->ev_join);
+    if (c->st2) cudaStreamDestroy(c->st2);
     for (float * p : c->pools) cudaFree(p);
     for (float * p : { c->XS, c->VF }) cudaFree(p);
     for (float * p : { c->Y2, c->U, c->XC, c->keep, c->scan_sb, c->scan_ac, c->sel_l, c->sel_sum, c->den, c->Xp, c->Ap, c->Yk, c->r_wt, c->r_sg, c->r_z }) cudaFree(p);
@@ -2205,7 +2405,12 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
         const bool par = m->block == BLOCK_PARALLEL;
         fl(&c->X, cap * m->E); fl(&c->Hn, cap * m->E * (par ? 2 : 1)); fl(&c->Y, cap * m->E);
         if (par) { fl(&c->Y2, cap * m->E); fl(&c->U, cap * m->E * 2); fl(&c->XC, cap * m->E * 2); }
-        else if (m->has_pair) fl(&c->Y2, cap * m->E);
+        else if (m->has_pair || m->block == BLOCK_SHARED) fl(&c->Y2, cap * m->E);
+        if (m->block == BLOCK_SHARED) {
+            fl(&c->F, cap * (size_t) m->max_dense); fl(&c->SZ, cap * (size_t) m->side_dim);
+            SCU(cudaStreamCreateWithFlags(&c->st2, cudaStreamNonBlocking));
+            SCU(cudaEventCreateWithFlags(&c->ev_fork, cudaEventDisableTiming)); SCU(cudaEventCreateWithFlags(&c->ev_join, cudaEventDisableTiming));
+        }
         if (m->depth_avg) fl(&c->keep, (m->layers.size() + 1) * cap * m->E);
         if (m->block == BLOCK_HYPER) fl(&c->XS, (size_t) m->streams * cap * m->E);
         if (m->vfirst_width > 0) fl(&c->VF, cap * (size_t) m->vfirst_width);
@@ -2236,7 +2441,7 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
         fl(&c->CV, cap * m->maxCV); fl(&c->BG, cap * m->maxBG); fl(&c->O, cap * m->maxA);
         fl(&c->rec, m->rec_floats);
         if (m->dtype == STACK_BF16) {
-            c->xb_elems = std::max(cap * (size_t) std::max({ 2 * m->E, m->maxA, m->maxOL, m->maxP }), moe_rows * (size_t) std::max(m->E, m->max_eff));
+            c->xb_elems = std::max(cap * (size_t) std::max({ 2 * m->E, m->maxA, m->maxOL, m->maxP, m->max_dense, m->side_dim }), moe_rows * (size_t) std::max(m->E, m->max_eff));
             SCU(cudaMalloc(&c->xb, c->xb_elems * 2));
             SCU(cudaMalloc(&c->xpart, umma_part_floats(c->sm_count) * 4));
         }
@@ -2337,7 +2542,7 @@ void stack_ctx_clear(StackCtx * c) {
     // recurrent state back to zero; cached positions need no clearing: a sequence only reads positions it wrote
     SCU(cudaMemsetAsync(c->rec, 0, std::max<size_t>(c->m->rec_floats, 4) * 4, c->st));
     SCU(cudaStreamSynchronize(c->st));
-    c->n_past = 0;
+    c->n_past = 0; c->last_token = -1;
     c->h_last = nullptr; c->d_last_row = -1;
 }
 
@@ -2362,7 +2567,7 @@ void stack_decode(StackCtx * c, const int32_t * tokens, int n, int pos0, const i
     ensure_logit_rows(c, std::max(n_rows, 1));
     SCU(cudaEventRecord(c->ev0, c->st));
     if (n == 1 && n_rows == 1 && !c->taps && graph_enabled() && !c->graph_failed) {
-        c->h_step->st.pos0 = pos0; c->h_step->st.n_tokens = 1; c->h_step->tokens[0] = tokens[0];
+        c->h_step->st = StepState{pos0, 1, c->last_token}; c->h_step->tokens[0] = tokens[0];
         if (!c->g_token) {
             SCU(cudaStreamSynchronize(c->st));
             const int64_t before = c->launches;
@@ -2394,7 +2599,7 @@ void stack_decode(StackCtx * c, const int32_t * tokens, int n, int pos0, const i
         for (int i0 = 0; i0 < n; i0 += c->cap) {
             const int T = std::min(c->cap, n - i0);
             SCU(cudaStreamSynchronize(c->st));              // the pinned header is free again
-            c->h_step->st.pos0 = pos0 + i0; c->h_step->st.n_tokens = T;
+            c->h_step->st = StepState{pos0 + i0, T, i0 ? tokens[i0 - 1] : c->last_token};
             std::memcpy(c->h_step->tokens, tokens + i0, (size_t) T * 4);
             int nr = 0;
             while (ri < n_rows && rows[ri] < i0 + T) c->h_step->rows[nr++] = rows[ri++] - i0;
@@ -2411,7 +2616,7 @@ void stack_decode(StackCtx * c, const int32_t * tokens, int n, int pos0, const i
         if (row_off) { c->d_last_row = row_off - 1; c->h_last = c->h_logits + (size_t) (row_off - 1) * m.vocab; }
     }
     cudaEventElapsedTime(&c->last_ms, c->ev0, c->ev1);
-    c->n_past = pos0 + n;
+    c->n_past = pos0 + n; c->last_token = tokens[n - 1];
     if (logits_out && n_rows > 0) std::memcpy(logits_out, c->h_logits, (size_t) n_rows * m.vocab * 4);
 }
 
@@ -2433,7 +2638,7 @@ void stack_generate_greedy(StackCtx * c, int32_t first_token, int pos0, int n_st
     SCU(cudaSetDevice(m.device));
     ensure_logit_rows(c, 1);
     SCU(cudaStreamSynchronize(c->st));
-    c->h_step->st.pos0 = pos0; c->h_step->st.n_tokens = 1; c->h_step->tokens[0] = first_token;
+    c->h_step->st = StepState{pos0, 1, c->last_token}; c->h_step->tokens[0] = first_token;
     const auto body = [&]() {
         enqueue_layers(c, 1);
         enqueue_head(c, 1, 0, true);
@@ -2464,7 +2669,7 @@ void stack_generate_greedy(StackCtx * c, int32_t first_token, int pos0, int n_st
     SCU(cudaStreamSynchronize(c->st));
     cudaEventElapsedTime(&c->last_ms, c->ev0, c->ev1);
     c->launches += c->n_greedy_launches * n_steps;
-    c->n_past = pos0 + n_steps;
+    c->n_past = pos0 + n_steps; c->last_token = n_steps > 1 ? out_tokens[n_steps - 2] : first_token;      // the newest token that went through the layers
     c->d_last_row = 0; c->h_last = nullptr;       // the last token's logits are on the device only
 }
 

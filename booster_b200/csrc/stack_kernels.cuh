@@ -50,6 +50,7 @@ template <int VEC> __device__ __forceinline__ void st_chunk(float * p, const flo
 struct StepState {
     int32_t pos0;       // position of the step's first token within its sequence
     int32_t n_tokens;
+    int32_t prev;       // the token before the step's first (-1: there is none)
 };
 
 // ---- RMS norm of one group by one warp: y = x / sqrt(mean(x^2) + eps) * w ------------------------------------------------
@@ -1769,6 +1770,7 @@ __global__ void __launch_bounds__(1024) k_argmax_advance(const float * __restric
         if (idx == 0x7fffffff) idx = 0;
         out[*counter] = idx;
         *counter += 1;
+        st->prev = *token_slot;
         *token_slot = idx;
         st->pos0 += 1;
     }

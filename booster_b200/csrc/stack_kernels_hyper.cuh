@@ -235,14 +235,14 @@ __device__ __forceinline__ float gqa_score(const GqaScore & sc, float dot, float
 // blocks of blockIdx.z walk its keys (block means first, then tokens) in alternating chunks of 32: a lane per key for the score,
 // a lane per 32nd value channel for the weighted sum, a running maximum and denominator per warp. The query's warps merge in
 // shared memory, the blocks through `part`, merged by the block that finishes last (an atomic counter, no waiting). The sink
-// joins the denominator once at the very end; the output is multiplied by sigmoid(gate[t][h]) when a gate is given.
+// joins the denominator once at the very end; the output is multiplied by sigmoid(gate) when a gate is given (one per head, or one per entry).
 struct GqaAttnArgs {
     const float * Q; int ldq;
     const float * cache; const float * pool; int ldc;
     const StepState * st;
     float * A;                                  // [T][H x V]
     const float * r1; const float * r2; const float * sink;      // [H] each; r1 == nullptr: no penalty; sink == nullptr: none
-    const float * gate; int ldg;                // gate pre-activations, one per head, rows of stride ldg (nullptr: none)
+    const float * gate; int ldg, gate_per_entry; // gate pre-activations, rows of stride ldg: one per head, or one per entry of A[t] (nullptr: none)
     int T, H, G, D, V;
     GqaScore sc;
     GqaMask mask;
@@ -262,7 +262,12 @@ __global__ void __launch_bounds__(256) k_gqa_attn(const GqaAttnArgs a) {
     // asked for together with the queries (one round trip to memory, not one each): the step's position and the head's constants
     const int pos0 = a.st->pos0;
     const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r1 ? a.r2[h] : 0.f, snk = a.sink ? a.sink[h] : 0.f;
-    const float gate_in = a.gate && t < a.T ? a.gate[(size_t) t * a.ldg + h] : 0.f;
+    float gate_in[VPL];                                     // of this lane's value channels
+#pragma unroll
+    for (int i = 0; i < VPL; i++) {
+        const int vi = lane + 32 * i;
+        gate_in[i] = a.gate && t < a.T && vi < a.V ? a.gate[(size_t) t * a.ldg + (a.gate_per_entry ? h * a.V + vi : h)] : 0.f;
+    }
     for (int i = tid; i < a.TQ * a.D; i += 256) {
         const int q = i / a.D, e = i - q * a.D;
         qs[i] = t0 + q < a.T ? a.Q[(size_t) (t0 + q) * a.ldq + (size_t) h * a.D + e] : 0.f;
@@ -372,9 +377,8 @@ __global__ void __launch_bounds__(256) k_gqa_attn(const GqaAttnArgs a) {
         l = fmaf(l, f, expf(snk - mm));
     }
     f /= l;
-    if (a.gate) f *= sigmoidf_(gate_in);
 #pragma unroll
-    for (int i = 0; i < VPL; i++) if (lane + 32 * i < a.V) a.A[(size_t) t * a.H * a.V + (size_t) h * a.V + lane + 32 * i] = acc[i] * f;
+    for (int i = 0; i < VPL; i++) if (lane + 32 * i < a.V) a.A[(size_t) t * a.H * a.V + (size_t) h * a.V + lane + 32 * i] = a.gate ? acc[i] * f * sigmoidf_(gate_in[i]) : acc[i] * f;
 }
 
 // Prompt portions run the same attention as float32 products around a row soft-max, like the other attentions of the family:

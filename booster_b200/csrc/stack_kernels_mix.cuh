@@ -403,19 +403,20 @@ __global__ void k_sig_weight_rows(float * __restrict__ S, int n_rows, int G, int
     const float sl = slope[h], b = pb[h];
     for (int n = lane; n < nk; n += 32) s[n] = (t < T && n <= p) ? sigmoidf_(fmaf(s[n], scale, b - sl * (float) (p - n))) : 0.f;
 }
-// Or[g][Tpad][R][V] -> A[t][h][V], times sigmoid(gate[t][h]) when a gate is given (one number per head, rows of stride ldg)
-__global__ void k_group_o_layout(const float * __restrict__ Or, int Tpad, int H, int G, int V, float * __restrict__ A, const float * __restrict__ gate = nullptr, int ldg = 0) {
+// Or[g][Tpad][R][V] -> A[t][h][V], times sigmoid(gate[t][h]) when a gate is given (one number per head, or per_entry = 1: one per entry of
+// A[t]; rows of stride ldg)
+__global__ void k_group_o_layout(const float * __restrict__ Or, int Tpad, int H, int G, int V, float * __restrict__ A, const float * __restrict__ gate = nullptr, int ldg = 0, int per_entry = 0) {
     const int t = blockIdx.x, R = H / G;
     for (int i = threadIdx.x; i < H * V; i += blockDim.x) {
         const int h = i / V, d = i - h * V, g = h / R, hq = h - g * R;
         const float o = Or[(((size_t) g * Tpad + t) * R + hq) * V + d];
-        A[(size_t) t * H * V + i] = gate ? o * sigmoidf_(gate[(size_t) t * ldg + h]) : o;
+        A[(size_t) t * H * V + i] = gate ? o * sigmoidf_(gate[(size_t) t * ldg + (per_entry ? i : h)]) : o;
     }
 }
 
 // ---- routed mixture of gated units --------------------------------------------------------------------------------------------------
-// Router, per token, in float32: z = W_r h, s = softmax(z) over all n experts (score_fn 0) or s_i = sigmoid(z_i), each expert by
-// itself (score_fn 1). Choices go by c = s + corr (corr == nullptr: c = s). The expert list is cut into n_groups consecutive blocks
+// Router, per token, in float32: z = W_r h (+ bias), s = softmax(z) over all n experts (score_fn 0) or s_i = sigmoid(z_i), each expert by
+// itself (score_fn 1), or s = z (score_fn 2: the choice goes by the logits and weighs in with the soft-max among the chosen ones). Choices go by c = s + corr (corr == nullptr: c = s). The expert list is cut into n_groups consecutive blocks
 // of equal size; a block ranks by the best c inside it and the choice is confined to the `keep` best-ranked blocks: of their experts
 // the `top` with the largest c are taken (lowest index first among equals). A choice weighs in with s * scale as it is, or, with
 // `norm_w`, with s * scale over the sum of the chosen s (+ 1e-20).
@@ -431,10 +432,11 @@ struct RouteArgs {
     float scale;
     int32_t * sel; float * wt; float * sg;
     float * z; int * counter;
-    int score_fn;       // 0: soft-max over the experts; 1: sigmoid of each logit
+    int score_fn;       // 0: soft-max over the experts; 1: sigmoid of each logit; 2: the logits, soft-max over the chosen
     int wpr;            // warps per router row: 1 (a block takes 8 rows) or 8 (a block takes one row, each warp an eighth of it: steps of few tokens)
     const float * corr = nullptr;
     int norm_w = 0;
+    const float * bias = nullptr;      // added to the logits
 };
 __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
     extern __shared__ float rsm[];
@@ -465,7 +467,7 @@ __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
             acc = 0.f;
             for (int k = 0; k < wpr; k++) acc += psum[k];
         }
-        if (lane == 0 && kw == 0) { if (e < a.n) z[e] = acc; else a.sg[t] = sigmoidf_(acc); }
+        if (lane == 0 && kw == 0) { if (e < a.n) z[e] = a.bias ? acc + a.bias[e] : acc; else a.sg[t] = sigmoidf_(acc); }
     }
     if (gridDim.y > 1) {
         __threadfence();
@@ -480,6 +482,8 @@ __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
     const int per = a.n / a.n_groups;
     if (a.score_fn == 1) {
         for (int i = lane; i < a.n; i += 32) { s[i] = sigmoidf_(__ldcg(z + i)); elig[i] = -INFINITY; }
+    } else if (a.score_fn == 2) {
+        for (int i = lane; i < a.n; i += 32) { s[i] = __ldcg(z + i); elig[i] = -INFINITY; }
     } else {
         float mx = -INFINITY;
         for (int i = lane; i < a.n; i += 32) { const float v = __ldcg(z + i); s[i] = v; mx = fmaxf(mx, v); }
@@ -511,7 +515,7 @@ __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
         }
         __syncwarp();
     }
-    float chosen = 0.f;
+    float chosen = 0.f, z0 = -INFINITY, z1 = -INFINITY, zmax = -INFINITY;      // score_fn 2: the logits of choices lane and lane + 32, the largest one
     for (int r = 0; r < a.top; r++) {
         float bv = -INFINITY; int bi = 0x7fffffff;
         for (int i = lane; i < a.n; i += 32) if (elig[i] > bv) { bv = elig[i]; bi = i; }
@@ -520,10 +524,18 @@ __global__ void __launch_bounds__(256) k_moe_route(const RouteArgs a) {
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
         const float w = bi == 0x7fffffff ? 0.f : s[bi];    // none left: fewer eligible experts than `top` (refused at load), or a score that is no number: a slot of weight 0
+        if (a.score_fn == 2 && bi != 0x7fffffff) { if (r == 0) zmax = w; if (r == lane) z0 = w; if (r == lane + 32) z1 = w; }
         if (bi == 0x7fffffff) bi = 0;
         chosen += w;
         if (lane == 0) { a.sel[t * a.top + r] = bi; a.wt[t * a.top + r] = w * a.scale; elig[bi] = -INFINITY; }
         __syncwarp();
+    }
+    if (a.score_fn == 2) {
+        const float e0 = z0 == -INFINITY ? 0.f : expf(z0 - zmax), e1 = z1 == -INFINITY ? 0.f : expf(z1 - zmax);
+        const float f = a.scale / warp_sum(e0 + e1);
+        if (lane < a.top) a.wt[t * a.top + lane] = e0 == 0.f ? 0.f : e0 * f;
+        if (lane + 32 < a.top) a.wt[t * a.top + lane + 32] = e1 == 0.f ? 0.f : e1 * f;
+        return;
     }
     if (a.norm_w) {
         const float f = 1.0f / (chosen + 1e-20f);
