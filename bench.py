@@ -346,6 +346,27 @@ def bench_kogerax(args):
     return 0
 
 
+def bench_bozisun(args):
+    """`--family stack --stack-design bozisun`: prefill and decode throughput of the Bozisun design (bfloat16 weights; random) at sizes
+    resembling real layers, beside the closest existing model, the Rumurax design (the same soft-max attention over grouped heads, a
+    routed mixture of silu units), at equal width / layers / heads / vocabulary and with as many feed-forward units read per token.
+    Comparable figures: the decode fraction of the measured HBM bandwidth and the prefill rate in weight bytes x tokens per second."""
+    from booster_b200 import _lib, engine, stack_io
+    L = _lib.lib()
+    hbm, hbm_src = peaks()
+    out = {"family": "stack", "design": "Bozisun", "closest": "Rumurax", "dtype": "bf16", "data": "synthetic (random bfloat16 weights)", "hbm_gbs_peak": hbm,
+           "hbm_peak_source": hbm_src, "steps": args.steps, "warmup": args.warmup, "sizes": {}}
+    for name, sz in STACK_SIZES.items():
+        if args.stack_size and name != args.stack_size:
+            continue
+        res = {}
+        res["bozisun"] = time_stack_model(engine, L, stack_io, stack_io.bozisun_config(**sz), os.path.join(MODEL_DIR, f"bozisun_{name}_s1234"), args, hbm)
+        res["rumurax"] = time_stack_model(engine, L, stack_io, stack_io.rumurax_config(**sz), os.path.join(MODEL_DIR, f"rumurax_{name}_s1234"), args, hbm)
+        out["sizes"][name] = res
+    print(json.dumps(out))
+    return 0
+
+
 def bench_stack(args):
     """Prefill and decode throughput of the Matulorn design (bfloat16 weights; random) at sizes resembling real layers, the
     LLaMA path (Q8_0, the closest block format in bytes per weight) at equal width / ff / layers / vocabulary beside it, and
@@ -451,11 +472,11 @@ def main():
     ap.add_argument("--family", default="llama", choices=["llama", "stack"],
                     help="stack: the layer-stack family (Matulorn design) beside the LLaMA path at equal layer sizes; the default workload is untouched")
     ap.add_argument("--stack-size", default="", choices=[""] + sorted(STACK_SIZES), help="--family stack: one size only")
-    ap.add_argument("--stack-design", default="matulorn", choices=["matulorn", "dopilorn", "tosevik", "rumurax", "kogerax"],
-                    help="--family stack: which design is measured (matulorn beside the LLaMA path; dopilorn beside matulorn; tosevik beside dopilorn; rumurax beside tosevik; kogerax beside tosevik)")
+    ap.add_argument("--stack-design", default="matulorn", choices=["matulorn", "dopilorn", "tosevik", "rumurax", "kogerax", "bozisun"],
+                    help="--family stack: which design is measured (matulorn beside the LLaMA path; dopilorn beside matulorn; tosevik beside dopilorn; rumurax beside tosevik; kogerax beside tosevik; bozisun beside rumurax)")
     args = ap.parse_args()
     if args.family == "stack":
-        return {"matulorn": bench_stack, "dopilorn": bench_dopilorn, "tosevik": bench_tosevik, "rumurax": bench_rumurax, "kogerax": bench_kogerax}[args.stack_design](args)
+        return {"matulorn": bench_stack, "dopilorn": bench_dopilorn, "tosevik": bench_tosevik, "rumurax": bench_rumurax, "kogerax": bench_kogerax, "bozisun": bench_bozisun}[args.stack_design](args)
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))

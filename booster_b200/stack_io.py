@@ -1,4 +1,4 @@
-"""Synthetic models of the layer-stack family (Matulorn, Dopilorn, Tosevik, Rumurax and Kogerax designs; config.json + model.safetensors) for benchmarks and smoke runs: random
+"""Synthetic models of the layer-stack family (Matulorn, Dopilorn, Tosevik, Rumurax, Kogerax and Bozisun designs; config.json + model.safetensors) for benchmarks and smoke runs: random
 bfloat16 weights of the right shapes, the counterpart of gguf_io.synth_llama for the GGUF path. Pure host code."""
 from __future__ import annotations
 
@@ -123,6 +123,51 @@ def kogerax_config(width: int, n_layer: int, ff: int, heads: int, vocab: int = 3
                                                           "router": {"experts": experts, "identity": identity, "top": top}}
         layers.append({"type": kind, "mixer": mx, "mlp": mlp})
     return {"architecture": "Kogerax", "embedding": {"scale": float(width) ** 0.5}, "layers": layers, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "vocab": vocab, "width": width}
+
+
+def bozisun_config(width: int, n_layer: int, ff: int, heads: int, vocab: int = 32000, head_dim: int = 128, kv_heads: int = 0, experts: int = 16, top: int = 4,
+                   side_dim: int = 0, buckets: int = 65521, loop=(1, 3, 2)) -> dict:
+    """a Bozisun configuration whose layers resemble a real model's: dense feed-forwards and, on every second layer, a routed mixture whose
+    chosen experts are as wide together as a dense one; token inputs of width / 16; layers loop[0] .. loop[1] - 1 run loop[2] times"""
+    e_ff = max(8, ff // top // 8 * 8)
+    layers = []
+    for i in range(n_layer):
+        mx = {"heads": heads, "kv_heads": kv_heads or max(1, heads // 4), "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+              "rot": {"base": 500000.0, "dims": head_dim // 2, "scaling": {"factor": 8.0, "fast": 32.0, "slow": 1.0, "original": 4096}}}
+        mlp = {"kind": "moe", "expert": {"ff": e_ff}, "router": {"experts": experts, "top": top}} if i % 2 else {"kind": "dense", "ff": ff}
+        layers.append({"type": "attention", "mixer": mx, "mlp": mlp})
+    cfg = {"architecture": "Bozisun", "embedding": {"bigram": {"buckets": buckets, "mul_prev": 1009, "mul_cur": 31}}, "layers": layers, "logit_softcap": 50.0,
+           "norm": {"eps": 1e-6}, "token_side": {"dim": side_dim or max(8, width // 16)}, "vocab": vocab, "width": width}
+    if loop and loop[1] <= n_layer:
+        cfg["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return cfg
+
+
+def bozisun_shapes(cfg: dict) -> Dict[str, List[int]]:
+    E, V, n = cfg["width"], cfg["vocab"], len(cfg["layers"])
+    t: Dict[str, List[int]] = {"embed": [V, E]}
+    bg, sd = (cfg.get("embedding") or {}).get("bigram"), (cfg.get("token_side") or {}).get("dim", 0)
+    if bg:
+        t["bigram"] = [bg["buckets"] + 1, E]
+    if sd:
+        t["side.embed"] = [V, n * sd]
+    for i, L in enumerate(cfg["layers"]):
+        p, mx, mj = f"l{i}.", L["mixer"], L.get("mlp")
+        H, D, Vd, m = mx["heads"], mx["dim"], mx["vdim"], p + "mix."
+        G = mx.get("kv_heads", H)
+        t.update({p + "norm1": [E], m + "q": [H * D, E], m + "k": [G * D, E], m + "v": [G * Vd, E], m + "q.norm": [D], m + "k.norm": [D], m + "g": [H * Vd, E], m + "o": [E, H * Vd]})
+        if mj and mj["kind"] == "dense":
+            t.update({p + "mlp.gate": [mj["ff"], E], p + "mlp.up": [mj["ff"], E], p + "mlp.down": [E, mj["ff"]]})
+        elif mj:
+            f = mj["expert"]["ff"]
+            for e in range(mj["router"]["experts"]):
+                t.update({f"{p}mlp.e{e}.gate": [f, E], f"{p}mlp.e{e}.up": [f, E], f"{p}mlp.e{e}.down": [E, f]})
+            t.update({p + "mlp.router": [mj["router"]["experts"], E], p + "mlp.router.b": [mj["router"]["experts"]]})
+        if sd:
+            t.update({p + "side.gate": [sd, E], p + "side.proj": [E, sd], p + "side.norm": [E]})
+    t["final.norm"] = [E]
+    t["head"] = [V, E]
+    return t
 
 
 def rumurax_shapes(cfg: dict) -> Dict[str, List[int]]:
@@ -296,6 +341,8 @@ def tensor_shapes(cfg: dict) -> Dict[str, List[int]]:
         return rumurax_shapes(cfg)
     if cfg.get("architecture") == "Kogerax":
         return kogerax_shapes(cfg)
+    if cfg.get("architecture") == "Bozisun":
+        return bozisun_shapes(cfg)
     E, V = cfg["width"], cfg["vocab"]
     t = {"embed": [V, E]}
     for i, L in enumerate(cfg["layers"]):
