@@ -235,6 +235,8 @@ struct StackCtx {
     cudaStream_t st2 = nullptr;           // BLOCK_SHARED, few-token steps: the feed-forward beside the mixer
     cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
     float * F = nullptr, * SZ = nullptr;  // BLOCK_SHARED: units of a dense feed-forward [cap][max_dense]; the token input's gate [cap][side_dim]
+    float * XE = nullptr;                 // few-token steps: the summed rows in front of the token input
+    int * end_counter = nullptr;          // per token: blocks of the layer's last launch done
     float * XS = nullptr, * VF = nullptr; // hyper-connections: the streams [S][cap][E]; value mixing: the first mixing layer's values of this pass [cap][G V]
     std::vector<float *> pools;           // per attention cache: means of whole blocks of cached rows (nullptr: the layer keeps none)
     float * Y2 = nullptr, * U = nullptr, * XC = nullptr;     // parallel blocks: the feed-forward's output, the convolved inputs [2][cap][E], [x; x0] rows
@@ -1395,12 +1397,13 @@ bool simt_big_enabled() {
 }
 // float32 product on the CUDA cores with explicit operand layout (the attention's two products over cached rows)
 // A second batch level (nz2 products per first-level index, strides sX2 / sW2 / sY2) serves operands that are cut twice: tiles x heads.
+struct See { int rows = 0, pos = 0, step = 0; };      // LinArgs::see_*
 void gemm_f32(StackCtx * c, const float * X, int ldx, long long sX, const float * W, int w_kn, int ldw, long long sW, float * Y, int ldy, long long sY,
-              int M, int N, int K, int batch, int nz2 = 1, long long sX2 = 0, long long sW2 = 0, long long sY2 = 0, int accum = 0) {
+              int M, int N, int K, int batch, int nz2 = 1, long long sX2 = 0, long long sW2 = 0, long long sY2 = 0, int accum = 0, See see = See()) {
     const auto al16 = [](const void * p) { return ((uintptr_t) p & 15) == 0; };
     LinArgs a{X, W, nullptr, Y, M, N, K, ldx, ldy, sX, sW, sY, 0, 0, 0.f, 0.f, w_kn, ldw, nz2, sX2, sW2, sY2};
     a.vec = K % 4 == 0 && ldx % 4 == 0 && sX % 4 == 0 && sW % 4 == 0 && sX2 % 4 == 0 && sW2 % 4 == 0 && ldw % 4 == 0 && al16(X) && al16(W);
-    a.accum = accum;
+    a.accum = accum; a.see_rows = see.rows; a.see_pos = see.pos; a.see_step = see.step;
     if (a.vec && M >= SG_BM && N >= SG_BN && simt_big_enabled())       // operands that fill 128 x 128 tiles
         k_gemm_simt_big<<<dim3((unsigned) ((N + SG_BN - 1) / SG_BN), (unsigned) ((M + SG_BM - 1) / SG_BM), (unsigned) (batch * nz2)), 256, 0, c->st>>>(a);
     else k_gemm_simt<float><<<dim3((unsigned) ((N + 63) / 64), (unsigned) ((M + 63) / 64), (unsigned) (batch * nz2)), 256, 0, c->st>>>(a);
@@ -1793,6 +1796,20 @@ bool gqa_tiles_enabled() {
     return on;
 }
 
+bool gqg_enabled() {
+    static const bool on = [] { const char * e = std::getenv("BOOSTER_B200_STACK_GQA_GROUP"); return !(e && e[0] == '0'); }();
+    return on;
+}
+// few-token steps: the kernel that takes a key/value head's queries together reads whole 16-byte chunks (every cached row is a multiple of 4
+// floats then; the caches' bases are 16-byte aligned plus whole rows)
+bool gqg_usable(const LayerSpec & L) { return L.D % 4 == 0 && L.V % 4 == 0 && L.D <= 256 && L.V <= 256 && gqg_enabled(); }
+int gqg_heads(const LayerSpec & L) {      // query heads a block takes: a power of two, up to 8 (4 beyond 128 entries per head)
+    const int R = L.H / L.KH, most = L.D > 128 || L.V > 128 ? 4 : 8;
+    int n = 1;
+    while (n < R && n < most) n *= 2;
+    return n;
+}
+
 // soft-max attention over grouped heads: P[t] = [ q | k | v | output gates ] -> per-head norms, rotation, value mixing; keys and
 // values to the cache row of the token's position (and the means of the blocks this step completes to the pool) -> attention
 // under the layer's mask -> gate -> output product
@@ -1829,14 +1846,16 @@ void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
             const float * keys = cache + jlo * row;
             const long long sK = masked ? (long long) TQ * row : 0;
             const long long grp = (long long) ng * M * ld;
-            gemm_f32(c, c->QK + (size_t) g0 * M * D, D, (long long) M * D, keys, 0, row, sK, c->att_scores + npc, ld, (long long) M * ld, M, nk, D, ng,
-                     G, (long long) Tpad * Rh * D, D, grp);
+            if (masked) gemm_f32(c, c->QK + (size_t) g0 * M * D, D, (long long) M * D, keys, 0, row, sK, c->att_scores + npc, ld, (long long) M * ld, M, nk, D, ng,
+                                 G, (long long) Tpad * Rh * D, D, grp);
+            else gemm_f32(c, c->QK + (size_t) g0 * M * D, D, 0, keys, 0, row, 0, c->att_scores, ld, 0, ng * M, nk, D, 1,      // all tiles meet the same keys: one tall operand
+                          G, (long long) Tpad * Rh * D, D, grp, 0, See{Rh, pos0 + g0 * TQ, 0});
             if (npc) gemm_f32(c, c->QK + (size_t) g0 * M * D, D, (long long) M * D, pool, 0, row, 0, c->att_scores, ld, (long long) M * ld, M, npc, D, ng,
                               G, (long long) Tpad * Rh * D, D, grp);
             const int rows = ng * M * G;
             k_gqa_softmax_rows<<<(rows + 7) / 8, 256, 0, c->st>>>(c->att_scores, ng * M, G, Rh, TQ, npc, nk, span, mask, sc, L.r1, L.r2, L.sink, st, g0, T);
             gemm_f32(c, c->att_scores + npc, ld, (long long) M * ld, keys + (size_t) G * D, 1, row, sK, c->OL + (size_t) g0 * M * V, V, (long long) M * V, M, V, nk, ng,
-                     G, grp, V, (long long) Tpad * Rh * V);
+                     G, grp, V, (long long) Tpad * Rh * V, 0, masked ? See() : See{Rh, pos0 + g0 * TQ, TQ});
             if (npc) gemm_f32(c, c->att_scores, ld, (long long) M * ld, pool + (size_t) G * D, 1, row, 0, c->OL + (size_t) g0 * M * V, V, (long long) M * V, M, V, npc, ng,
                               G, grp, V, (long long) Tpad * Rh * V, 1);
             c->launches++;
@@ -1846,12 +1865,27 @@ void mixer_gqattn(StackCtx * c, const LayerSpec & L, const RunSpec & R, int T) {
         linear(c, c->A, H * V, L.o, c->out, E, T);
         return;
     }
+    GqaAttnArgs a{c->CV, nq, cache, pool, row, st, c->A, L.r1, L.r2, L.sink, gate, ldp, gate_per_entry, T, H, G, D, V, sc, mask, 1, 1, 1, c->da_part, c->da_counter};
+    const int max_keys = L.mask_kind == MASK_CAUSAL ? c->n_ctx : std::min(c->n_ctx, L.window + (L.pool > 0 ? c->n_ctx / L.pool : 0));
+    if (T < 8 && gqg_usable(L)) {
+        const int RT = gqg_heads(L), ngrp = (H / G + RT - 1) / RT;
+        const int nsplit = std::max(1, std::min({ 2 * c->sm_count / (T * G * ngrp), (max_keys + 31) / 32, GQG_MAX_SPLIT }));
+        const dim3 grid((unsigned) T, (unsigned) (G * ngrp), (unsigned) nsplit);
+        const size_t smem = gqg_smem(RT, V);
+        const bool wide = D > 128 || V > 128;
+        if (RT == 1) { if (wide) k_gqa_attn_group<1, 2><<<grid, 256, smem, c->st>>>(a); else k_gqa_attn_group<1, 1><<<grid, 256, smem, c->st>>>(a); }
+        else if (RT == 2) { if (wide) k_gqa_attn_group<2, 2><<<grid, 256, smem, c->st>>>(a); else k_gqa_attn_group<2, 1><<<grid, 256, smem, c->st>>>(a); }
+        else if (RT == 4) { if (wide) k_gqa_attn_group<4, 2><<<grid, 256, smem, c->st>>>(a); else k_gqa_attn_group<4, 1><<<grid, 256, smem, c->st>>>(a); }
+        else k_gqa_attn_group<8, 1><<<grid, 256, smem, c->st>>>(a);
+        c->launches++;
+        linear(c, c->A, H * V, L.o, c->out, E, T);
+        return;
+    }
     const int TQ = T >= 4 ? 4 : T >= 2 ? 2 : 1, WPQ = 8 / TQ;
     const int blocks = ((T + TQ - 1) / TQ) * H;
-    const int max_keys = L.mask_kind == MASK_CAUSAL ? c->n_ctx : std::min(c->n_ctx, L.window + (L.pool > 0 ? c->n_ctx / L.pool : 0));
     const int nsplit = std::max(1, std::min({ 2 * c->sm_count / blocks, ((max_keys + 31) / 32 + WPQ - 1) / WPQ, GQA_MAX_SPLIT }));
-    const GqaAttnArgs a{c->CV, nq, cache, pool, row, st, c->A, L.r1, L.r2, L.sink, gate, ldp, gate_per_entry, T, H, G, D, V, sc, mask, TQ,
-                        (D % 4 == 0 && row % 4 == 0 && ((uintptr_t) cache & 15) == 0 && ((uintptr_t) pool & 15) == 0) ? 1 : 0, nsplit, c->da_part, c->da_counter};
+    a.TQ = TQ; a.nsplit = nsplit;
+    a.vec = (D % 4 == 0 && row % 4 == 0 && ((uintptr_t) cache & 15) == 0 && ((uintptr_t) pool & 15) == 0) ? 1 : 0;
     const dim3 grid((unsigned) ((T + TQ - 1) / TQ), (unsigned) H, (unsigned) nsplit);
     const int VPL = gqa_vpl(L);
     const size_t smem = ((size_t) TQ * D + (size_t) 8 * (2 + 32 * VPL)) * 4;
@@ -2185,16 +2219,20 @@ void layer_end(StackCtx * c, const LayerSpec & L, SumArgs a, const float * nw, i
     a.X = c->X; a.E = E; a.eps = m.eps; a.Hn = c->Hn;
     a.nw = dim > 0 ? nullptr : nw;
     const SideW s{m.side_table, (int) m.layers.size() * dim, L.side_off, dim, L.side_gate.w, L.side_proj.w, L.side_norm};
-    const size_t smem = end_smem(E, dim);
-    if (dim > 0 && T <= GEMV_MAX_T && smem <= 40 * 1024 && side_fused_enabled()) {
+    if (dim > 0 && T <= GEMV_MAX_T && E <= SIDE_MOST && dim <= SIDE_MOST && side_fused_enabled()) {
         const int vecw = m.dtype == STACK_F32 ? 4 : 8;
         int lpr = 1;                                       // lanes per row of the projection: as many as it has 16-byte pieces
         while (lpr < 32 && lpr * vecw < dim) lpr *= 2;
         a.nw = nw;
-        const dim3 grid(END_CTAS, (unsigned) T);
-        const auto go = [&](auto kernel) { kernel<<<grid, END_THREADS, smem, c->st>>>(a, s, c->d_step->tokens, m.vocab, end_slice(E), E % vecw == 0 ? 1 : 0, dim % vecw == 0 ? 1 : 0, lpr); };
-        if (m.dtype == STACK_F32) go(k_layer_end<float>); else go(k_layer_end<__nv_bfloat16>);
-        c->launches++;
+        const dim3 g1((unsigned) ((dim + SIDE_ROWS - 1) / SIDE_ROWS), (unsigned) T), g2((unsigned) ((E + side_rows_per_block(lpr) - 1) / side_rows_per_block(lpr)), (unsigned) T);
+        const auto go = [&](auto in, auto out) {
+            in<<<g1, SIDE_THREADS, (size_t) E * 4, c->st>>>(a, s, c->d_step->tokens, m.vocab, E % vecw == 0 ? 1 : 0, c->XE, c->SZ);
+            out<<<g2, SIDE_THREADS, (size_t) dim * 4, c->st>>>(a, s, c->XE, c->SZ, c->Y, c->end_counter, dim % vecw == 0 ? 1 : 0, lpr);      // Y: the mixer's output has been summed by then
+        };
+        if (m.dtype == STACK_F32) { if (E % 4 == 0) go(k_side_in<float>, k_side_out<float, 4>); else go(k_side_in<float>, k_side_out<float, 1>); }
+        else if (E % 4 == 0) go(k_side_in<__nv_bfloat16>, k_side_out<__nv_bfloat16, 4>);
+        else go(k_side_in<__nv_bfloat16>, k_side_out<__nv_bfloat16, 1>);
+        c->launches += 2;
         return;
     }
     if (E % 4 == 0) k_sum_join<4><<<T, nt, 0, c->st>>>(a);      // every buffer of a context is 16-byte aligned and its rows are E floats apart
@@ -2368,7 +2406,7 @@ void stack_ctx_free(StackCtx * c) {
     if (c->g_token) cudaGraphExecDestroy(c->g_token);
     if (c->g_greedy) cudaGraphExecDestroy(c->g_greedy);
     cudaFree(c->d_out_tokens); cudaFree(c->d_counter);
-    cudaFree(c->F); cudaFree(c->SZ);
+    cudaFree(c->F); cudaFree(c->SZ); cudaFree(c->XE); cudaFree(c->end_counter);
     if (c->ev_fork) cudaEventDestroy(c->ev_fork);
     if (c->ev_join) cudaEventDestroy(c->ev_join);
     if (c->st2) cudaStreamDestroy(c->st2);
@@ -2408,6 +2446,7 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
         else if (m->has_pair || m->block == BLOCK_SHARED) fl(&c->Y2, cap * m->E);
         if (m->block == BLOCK_SHARED) {
             fl(&c->F, cap * (size_t) m->max_dense); fl(&c->SZ, cap * (size_t) m->side_dim);
+            fl(&c->XE, (size_t) GEMV_MAX_T * m->E); fl((float **) &c->end_counter, GEMV_MAX_T);
             SCU(cudaStreamCreateWithFlags(&c->st2, cudaStreamNonBlocking));
             SCU(cudaEventCreateWithFlags(&c->ev_fork, cudaEventDisableTiming)); SCU(cudaEventCreateWithFlags(&c->ev_join, cudaEventDisableTiming));
         }
@@ -2490,6 +2529,7 @@ StackCtx * stack_ctx_new(StackModel * m, int n_ctx) {
             }
             if (L.kind == MIX_GQATTN) {       // key slices only while (tokens x heads x slices) stays under 8 per SM; one counter per (token, head) of a pass
                 da_part = std::max(da_part, (size_t) (8 * c->sm_count + 64) * (2 + 32 * (size_t) gqa_vpl(L)));
+                da_part = std::max(da_part, (size_t) (2 * c->sm_count + 8 * L.H) * 8 * (size_t) (2 + L.V));      // tokens x head groups x slices: two per SM, or one each
                 da_cnt = std::max(da_cnt, cap * (size_t) L.H);
                 continue;
             }

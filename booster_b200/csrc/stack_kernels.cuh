@@ -173,7 +173,13 @@ struct LinArgs {
     // k_gemv: entry z's input row is x_scale[z] times the row it reads (a routed expert that runs on a weighted input); no bias then
     const float * x_scale = nullptr;
     int accum = 0;      // k_gemm_simt only: Y += the product (a second set of keys joining a weighted sum)
+    // float32 tile kernels, see_rows > 0 (every earlier position is seen): row m of first-level entry z1 concerns positions 0 .. see_pos +
+    // z1 see_step + m / see_rows only. Positions are the columns (w_kn = 0: tiles beyond their rows' last one are left alone) or the inner
+    // dimension (w_kn = 1: the sum ends with the tile's last one, rounded up to 4; what lies up to there counts)
+    int see_rows = 0, see_pos = 0, see_step = 0;
 };
+// the last position a tile of rows m0 .. m0 + rows - 1 sees
+__device__ __forceinline__ int tile_sees(const LinArgs & a, int z1, int m0, int rows) { return a.see_pos + z1 * a.see_step + (min(m0 + rows, a.T) - 1) / a.see_rows; }
 enum { GLU_NONE = 0, GLU_SIGMOID = 1, GLU_GELU = 2 };
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, float alpha, float shift) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);      // limit = +inf: no clamp
@@ -297,6 +303,12 @@ __global__ void __launch_bounds__(256) k_gemm_simt(const LinArgs a) {
     const int z1 = blockIdx.z / a.nz2, z2 = blockIdx.z - z1 * a.nz2;
     const int r0 = a.seg ? a.seg[blockIdx.z] : 0, T = a.seg ? a.seg[blockIdx.z + 1] - r0 : a.T;
     if (m0 >= T) return;
+    int K = a.K;
+    if (a.see_rows > 0) {
+        const int last = tile_sees(a, z1, m0, 64);
+        if (a.w_kn) K = min(K, (last + 4) / 4 * 4);
+        else if (n0 > last) return;
+    }
     const float * X = a.seg ? a.X + (size_t) r0 * a.ldx : a.X + (size_t) z1 * a.sX + (size_t) z2 * a.sX2;
     const WT * W = reinterpret_cast<const WT *>(a.W) + (size_t) z1 * a.sW + (size_t) z2 * a.sW2;
     const int lr = tid >> 2, lk = (tid & 3) * 4;          // this thread stages 4 consecutive k of row lr
@@ -305,14 +317,14 @@ __global__ void __launch_bounds__(256) k_gemm_simt(const LinArgs a) {
     for (int i = 0; i < 4; i++)
 #pragma unroll
         for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
-    for (int k0 = 0; k0 < a.K; k0 += 16) {
+    for (int k0 = 0; k0 < K; k0 += 16) {
         {
             const int m = m0 + lr;
             float v[4] = { 0.f, 0.f, 0.f, 0.f };
             if (m < T) {
                 const float * p = X + (size_t) m * a.ldx + k0 + lk;
-                if (a.vec && k0 + lk + 3 < a.K) { const float4 f = *reinterpret_cast<const float4 *>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
-                else for (int i = 0; i < 4; i++) if (k0 + lk + i < a.K) v[i] = p[i];
+                if (a.vec && k0 + lk + 3 < K) { const float4 f = *reinterpret_cast<const float4 *>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+                else for (int i = 0; i < 4; i++) if (k0 + lk + i < K) v[i] = p[i];
             }
 #pragma unroll
             for (int i = 0; i < 4; i++) Xs[lk + i][lr] = v[i];
@@ -321,7 +333,7 @@ __global__ void __launch_bounds__(256) k_gemm_simt(const LinArgs a) {
             // [K][N] operand with 16-byte aligned rows: a thread takes 4 consecutive n of one k, the block one 16 x 64 tile
             const int kk = tid >> 4, n4 = (tid & 15) * 4, k = k0 + kk, n = n0 + n4;
             float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (k < a.K && n < a.N) {
+            if (k < K && n < a.N) {
                 const float * p = reinterpret_cast<const float *>(W) + (size_t) k * a.ldw + n;
                 if (n + 3 < a.N) f = *reinterpret_cast<const float4 *>(p);
                 else { f.x = p[0]; if (n + 1 < a.N) f.y = p[1]; if (n + 2 < a.N) f.z = p[2]; }
@@ -332,13 +344,13 @@ __global__ void __launch_bounds__(256) k_gemm_simt(const LinArgs a) {
             float v[4] = { 0.f, 0.f, 0.f, 0.f };
             if (n < a.N) {
                 if (a.w_kn) {
-                    for (int i = 0; i < 4; i++) if (k0 + lk + i < a.K) v[i] = wf(W, (size_t) (k0 + lk + i) * a.ldw + n);
+                    for (int i = 0; i < 4; i++) if (k0 + lk + i < K) v[i] = wf(W, (size_t) (k0 + lk + i) * a.ldw + n);
                 } else {
                     const size_t o = (size_t) n * (a.ldw > 0 ? a.ldw : a.K) + k0 + lk;
-                    if (sizeof(WT) == 4 && a.vec && k0 + lk + 3 < a.K) {
+                    if (sizeof(WT) == 4 && a.vec && k0 + lk + 3 < K) {
                         const float4 f = *reinterpret_cast<const float4 *>(reinterpret_cast<const float *>(W) + o);
                         v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-                    } else for (int i = 0; i < 4; i++) if (k0 + lk + i < a.K) v[i] = wf(W, o + i);
+                    } else for (int i = 0; i < 4; i++) if (k0 + lk + i < K) v[i] = wf(W, o + i);
                 }
             }
 #pragma unroll
@@ -393,6 +405,12 @@ __global__ void __launch_bounds__(256, 2) k_gemm_simt_big(const LinArgs a) {
     const float * X = a.X + (size_t) z1 * a.sX + (size_t) z2 * a.sX2;
     const float * W = reinterpret_cast<const float *>(a.W) + (size_t) z1 * a.sW + (size_t) z2 * a.sW2;
     const int ldw = a.ldw > 0 ? a.ldw : a.K;
+    int K = a.K;
+    if (a.see_rows > 0) {
+        const int last = tile_sees(a, z1, m0, SG_BM);
+        if (a.w_kn) K = min(K, (last + 4) / 4 * 4);
+        else if (n0 > last) return;
+    }
     float acc[8][8];
 #pragma unroll
     for (int i = 0; i < 8; i++)
@@ -408,23 +426,23 @@ __global__ void __launch_bounds__(256, 2) k_gemm_simt_big(const LinArgs a) {
         for (int h = 0; h < 2; h++) {
             const int m = m0 + lr + 64 * h;
             xr[h] = zero;
-            if (m < a.T && k0 + lk < a.K) xr[h] = *reinterpret_cast<const float4 *>(X + (size_t) m * a.ldx + k0 + lk);      // K is a multiple of 4
+            if (m < a.T && k0 + lk < K) xr[h] = *reinterpret_cast<const float4 *>(X + (size_t) m * a.ldx + k0 + lk);      // K is a multiple of 4
             wr[h] = zero;
             if (a.w_kn) {
                 const int k = k0 + kk + 8 * h, n = n0 + n4;
-                if (k < a.K && n < a.N) {
+                if (k < K && n < a.N) {
                     const float * p = W + (size_t) k * ldw + n;
                     if (n + 3 < a.N) wr[h] = *reinterpret_cast<const float4 *>(p);
                     else { wr[h].x = p[0]; if (n + 1 < a.N) wr[h].y = p[1]; if (n + 2 < a.N) wr[h].z = p[2]; }
                 }
             } else {
                 const int n = n0 + lr + 64 * h;
-                if (n < a.N && k0 + lk < a.K) wr[h] = *reinterpret_cast<const float4 *>(W + (size_t) n * ldw + k0 + lk);
+                if (n < a.N && k0 + lk < K) wr[h] = *reinterpret_cast<const float4 *>(W + (size_t) n * ldw + k0 + lk);
             }
         }
     };
     fetch(0);
-    for (int k0 = 0; k0 < a.K; k0 += SG_BK) {
+    for (int k0 = 0; k0 < K; k0 += SG_BK) {
 #pragma unroll
         for (int h = 0; h < 2; h++) {
             const float xv[4] = { xr[h].x, xr[h].y, xr[h].z, xr[h].w };
@@ -438,7 +456,7 @@ __global__ void __launch_bounds__(256, 2) k_gemm_simt_big(const LinArgs a) {
             }
         }
         __syncthreads();
-        if (k0 + SG_BK < a.K) fetch(k0 + SG_BK);
+        if (k0 + SG_BK < K) fetch(k0 + SG_BK);
 #pragma unroll
         for (int k = 0; k < SG_BK; k++) {
             const float4 x0 = *reinterpret_cast<const float4 *>(&Xs[k][ty * 4]), x1 = *reinterpret_cast<const float4 *>(&Xs[k][64 + ty * 4]);

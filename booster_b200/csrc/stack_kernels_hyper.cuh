@@ -381,12 +381,195 @@ __global__ void __launch_bounds__(256) k_gqa_attn(const GqaAttnArgs a) {
     for (int i = 0; i < VPL; i++) if (lane + 32 * i < a.V) a.A[(size_t) t * a.H * a.V + (size_t) h * a.V + lane + 32 * i] = a.gate ? acc[i] * f * sigmoidf_(gate_in[i]) : acc[i] * f;
 }
 
+// The same for heads whose queries share keys, in 16-byte loads (D, V multiples of 4, up to 256): a block takes one token and up to RT query
+// heads of one key/value head, so a cached row is fetched once for all of them. A warp walks strips of KS keys: all key and value rows of a
+// strip are asked for at once (a lane holds entries 4 lane .. 4 lane + 3 of every row, CH such chunks), the KS x RT dot products are summed
+// across the warp by halving (a lane ends with one (head, key) pair), and the weights go back by shuffles. The block's warps and the blocks
+// of blockIdx.z merge as above; blocks beyond what the sequence's length can fill (8 warps a strip each) leave at once.
+// grid (T, G x head groups, nsplit); part [T][gridDim.y][nsplit][RT][2 + V].
+constexpr int GQG_MAX_SPLIT = 64;
+inline size_t gqg_smem(int RT, int V) { return ((size_t) 8 * RT * (2 + V) + (size_t) RT * GQG_MAX_SPLIT) * 4; }
+template <int RT, int CH>
+__global__ void __launch_bounds__(256) k_gqa_attn_group(const GqaAttnArgs a) {
+    constexpr int KS = RT * CH > 4 ? 4 : 8, NV = KS * RT, REP = 32 / NV;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ int done_s;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t = blockIdx.x, R = a.H / a.G, ngrp = (R + RT - 1) / RT;
+    const int g = blockIdx.y / ngrp, h0 = g * R + (blockIdx.y - g * ngrp) * RT, nh = min(RT, (g + 1) * R - h0), V = a.V, MG = 2 + V;
+    const int pos0 = a.st->pos0, p = pos0 + t;
+    float4 q[RT][CH];
+#pragma unroll
+    for (int h = 0; h < RT; h++)
+#pragma unroll
+        for (int c = 0; c < CH; c++) {
+            const int e = 4 * lane + 128 * c;
+            q[h][c] = h < nh && e < a.D ? *reinterpret_cast<const float4 *>(a.Q + (size_t) t * a.ldq + (size_t) (h0 + h) * a.D + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    const int jlo = gqa_first_token(a.mask, p), nb = gqa_blocks_seen(a.mask, p), ntot = nb + p - jlo + 1, nstrip = (ntot + KS - 1) / KS;
+    const int ns = min((int) gridDim.z, (nstrip + 7) / 8), z = blockIdx.z;
+    if (z >= ns) return;
+    const int hh = lane / REP / KS, kk = lane / REP % KS;      // this lane's (head, key) of a strip
+    const bool mine = hh < nh;
+    const float r1 = a.r1 && mine ? a.r1[h0 + hh] : 0.f, r2 = a.r1 && mine ? a.r2[h0 + hh] : 0.f;
+    const float * tokens = a.cache + ((long long) jlo - nb) * a.ldc;
+    const size_t koff = (size_t) g * a.D, voff = (size_t) a.G * a.D + (size_t) g * V;
+    float4 acc[RT][CH];
+    float m = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int h = 0; h < RT; h++)
+#pragma unroll
+        for (int c = 0; c < CH; c++) acc[h][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = z * 8 + warp; s < nstrip; s += 8 * ns) {
+        const int n0 = s * KS;
+        float4 k[KS][CH], v[KS][CH];
+#pragma unroll
+        for (int i = 0; i < KS; i++) {
+            const int n = min(n0 + i, ntot - 1);               // past the end: the last row again, with weight 0
+            const float * row = n < nb ? a.pool + (size_t) n * a.ldc : tokens + (long long) n * a.ldc;
+#pragma unroll
+            for (int c = 0; c < CH; c++) {
+                const int e = 4 * lane + 128 * c;
+                k[i][c] = e < a.D ? __ldg(reinterpret_cast<const float4 *>(row + koff + e)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[i][c] = e < V ? __ldg(reinterpret_cast<const float4 *>(row + voff + e)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
+        float d[NV];
+#pragma unroll
+        for (int h = 0; h < RT; h++)
+#pragma unroll
+            for (int i = 0; i < KS; i++) {
+                float x = 0.f;
+#pragma unroll
+                for (int c = 0; c < CH; c++) x = fmaf(q[h][c].x, k[i][c].x, fmaf(q[h][c].y, k[i][c].y, fmaf(q[h][c].z, k[i][c].z, fmaf(q[h][c].w, k[i][c].w, x))));
+                d[h * KS + i] = x;
+            }
+        int o = 16;
+#pragma unroll
+        for (int n = NV; n > 1; n >>= 1, o >>= 1) {
+            const bool up = lane & o;
+#pragma unroll
+            for (int i = 0; i < NV / 2; i++) if (i < n / 2) {
+                const float send = up ? d[i] : d[i + n / 2], keep = up ? d[i + n / 2] : d[i];
+                d[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+        }
+#pragma unroll
+        for (; o > 0; o >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], o);
+        const int n = n0 + kk;
+        const float sc = n < ntot ? gqa_score(a.sc, d[0], r1, r2, n < nb ? 0 : p - (jlo + n - nb)) : -INFINITY;
+        float mx = sc;
+#pragma unroll
+        for (int b = REP; b < REP * KS; b <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, b));
+        const float mn = fmaxf(m, mx), corr = m == -INFINITY ? 0.f : expf(m - mn);      // the strip's first key is a real one: mn is finite
+        const float w = n < ntot ? expf(sc - mn) : 0.f;
+        float sum = w;
+#pragma unroll
+        for (int b = REP; b < REP * KS; b <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, b);
+        l = fmaf(l, corr, sum);
+        m = mn;
+#pragma unroll
+        for (int h = 0; h < RT; h++) {
+            const float f = __shfl_sync(0xffffffffu, corr, h * KS * REP);
+#pragma unroll
+            for (int c = 0; c < CH; c++) { acc[h][c].x *= f; acc[h][c].y *= f; acc[h][c].z *= f; acc[h][c].w *= f; }
+#pragma unroll
+            for (int i = 0; i < KS; i++) {
+                const float wk = __shfl_sync(0xffffffffu, w, (h * KS + i) * REP);
+#pragma unroll
+                for (int c = 0; c < CH; c++) {
+                    acc[h][c].x = fmaf(wk, v[i][c].x, acc[h][c].x); acc[h][c].y = fmaf(wk, v[i][c].y, acc[h][c].y);
+                    acc[h][c].z = fmaf(wk, v[i][c].z, acc[h][c].z); acc[h][c].w = fmaf(wk, v[i][c].w, acc[h][c].w);
+                }
+            }
+        }
+    }
+    // the block's warps: [8][RT][m, l, V sums]
+    float * fz = sm + (size_t) 8 * RT * MG;                    // [RT][GQG_MAX_SPLIT]
+    if (lane % (KS * REP) == 0) { float * o = sm + ((size_t) warp * RT + hh) * MG; o[0] = m; o[1] = l; }
+#pragma unroll
+    for (int h = 0; h < RT; h++)
+#pragma unroll
+        for (int c = 0; c < CH; c++) {
+            const int e = 4 * lane + 128 * c;
+            float * o = sm + ((size_t) warp * RT + h) * MG + 2 + e;
+            if (e < V) { *reinterpret_cast<float2 *>(o) = make_float2(acc[h][c].x, acc[h][c].y); *reinterpret_cast<float2 *>(o + 2) = make_float2(acc[h][c].z, acc[h][c].w); }
+        }
+    __syncthreads();
+    const size_t tg = (size_t) t * gridDim.y + blockIdx.y;
+    float * part = a.part + (tg * gridDim.z + z) * RT * MG;
+    const auto out = [&](int h, int e, float sum, float mm, float ll) {
+        float f = 1.0f;
+        if (a.sink) {                                          // exp(sink) joins the denominator: no key, no value
+            const float snk = a.sink[h0 + h], top = fmaxf(mm, snk);
+            f = expf(mm - top);
+            ll = fmaf(ll, f, expf(snk - top));
+        }
+        sum *= f / ll;
+        const int at = (h0 + h) * V + e;
+        if (a.gate) sum *= sigmoidf_(a.gate[(size_t) t * a.ldg + (a.gate_per_entry ? at : h0 + h)]);
+        a.A[(size_t) t * a.H * V + at] = sum;
+    };
+    for (int i = tid; i < nh * V; i += 256) {
+        const int h = i / V, e = i - h * V;
+        const float * o = sm + (size_t) h * MG;
+        float mm = -INFINITY, ll = 0.f, sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; w++) mm = fmaxf(mm, o[(size_t) w * RT * MG]);
+#pragma unroll
+        for (int w = 0; w < 8; w++) {
+            const float * ow = o + (size_t) w * RT * MG;
+            const float f = ow[0] == -INFINITY ? 0.f : expf(ow[0] - mm);
+            ll = fmaf(ow[1], f, ll);
+            sum = fmaf(ow[2 + e], f, sum);
+        }
+        if (ns == 1) out(h, e, sum, mm, ll);
+        else { part[h * MG + 2 + e] = sum; if (e == 0) { part[h * MG] = mm; part[h * MG + 1] = ll; } }
+    }
+    if (ns == 1) return;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) done_s = atomicAdd(a.counter + tg, 1) == ns - 1;
+    __syncthreads();
+    if (!done_s) return;
+    __threadfence();
+    if (tid == 0) a.counter[tg] = 0;
+    const float * ps = a.part + tg * gridDim.z * RT * MG;
+    for (int h = warp; h < nh; h += 8) {                       // every part's factor, and the head's maximum and denominator
+        float mz[2], lz[2];
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int y = lane + 32 * i;
+            mz[i] = y < ns ? __ldcg(ps + ((size_t) y * RT + h) * MG) : -INFINITY;
+            lz[i] = y < ns ? __ldcg(ps + ((size_t) y * RT + h) * MG + 1) : 0.f;
+        }
+        const float mm = warp_max(fmaxf(mz[0], mz[1]));
+        float ll = 0.f;
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const float f = mz[i] == -INFINITY ? 0.f : expf(mz[i] - mm);
+            fz[h * GQG_MAX_SPLIT + lane + 32 * i] = f;
+            ll = fmaf(lz[i], f, ll);
+        }
+        ll = warp_sum(ll);
+        if (lane == 0) { sm[(size_t) h * MG] = mm; sm[(size_t) h * MG + 1] = ll; }
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * V; i += 256) {
+        const int h = i / V, e = i - h * V;
+        float sum = 0.f;
+#pragma unroll 8
+        for (int y = 0; y < ns; y++) sum = fmaf(fz[h * GQG_MAX_SPLIT + y], __ldcg(ps + ((size_t) y * RT + h) * MG + 2 + e), sum);
+        out(h, e, sum, sm[(size_t) h * MG], sm[(size_t) h * MG + 1]);
+    }
+}
+
 // Prompt portions run the same attention as float32 products around a row soft-max, like the other attentions of the family:
 // per tile of TQ tokens and key/value head g, S = Q_g K_g^T (rows: the tile's tokens x the R = H / G query heads of the group),
 // this kernel turns scores into weights, then O = W V_g. A row of S holds [ npc columns of block means | nk columns of tokens ]:
 // token column n is position jlo + n with jlo = pos0 + tile TQ - span + 1 (span: the most tokens any row looks back, no more
 // than the sequence so far; the cache has a zero margin in front) or 0 when the products start at position 0 (span == 0).
-// S holds [g][n_rows = ng TQ R][npc + nk] for a group of ng tiles starting at tile0. One warp per row.
+// S holds [g][n_rows = ng TQ R][npc + nk] for a group of ng tiles starting at tile0. One warp per row. Without a mask (span == 0) columns
+// past the row's tile are neither computed nor read: weights are written up to the tile's last position, rounded up to 4.
 __global__ void k_gqa_softmax_rows(float * __restrict__ S, int n_rows, int G, int R, int TQ, int npc, int nk, int span, GqaMask mask, GqaScore sc,
                                    const float * __restrict__ r1v, const float * __restrict__ r2v, const float * __restrict__ sink,
                                    const StepState * __restrict__ st, int tile0, int T) {
@@ -395,7 +578,8 @@ __global__ void k_gqa_softmax_rows(float * __restrict__ S, int n_rows, int G, in
     const int g = id / n_rows, r = id - g * n_rows, h = g * R + r % R;
     const int t = tile0 * TQ + r / R, p = st->pos0 + t;
     float * s = S + (size_t) id * (npc + nk);
-    if (t >= T) { for (int n = lane; n < npc + nk; n += 32) s[n] = 0.f; return; }
+    const int nw = span > 0 ? npc + nk : min(npc + nk, npc + (st->pos0 + (t / TQ + 1) * TQ + 3) / 4 * 4);
+    if (t >= T) { for (int n = lane; n < nw; n += 32) s[n] = 0.f; return; }
     const int jlo = span > 0 ? st->pos0 + (t / TQ) * TQ - span + 1 : 0;
     const int n_lo = npc + gqa_first_token(mask, p) - jlo, n_hi = npc + p - jlo, nb = gqa_blocks_seen(mask, p);     // token columns n_lo .. n_hi, block columns 0 .. nb - 1
     const float r1 = r1v ? r1v[h] : 0.f, r2 = r1v ? r2v[h] : 0.f;
@@ -411,7 +595,7 @@ __global__ void k_gqa_softmax_rows(float * __restrict__ S, int n_rows, int G, in
     sum = warp_sum(sum);
     const float inv = 1.0f / (sum + (sink ? expf(snk - m) : 0.f));
     __syncwarp();                                           // the last pass walks the row from column 0: other lanes' columns
-    for (int n = lane; n < npc + nk; n += 32) s[n] = (n < nb || (n >= n_lo && n <= n_hi)) ? expf(s[n] - m) * inv : 0.f;
+    for (int n = lane; n < nw; n += 32) s[n] = (n < nb || (n >= n_lo && n <= n_hi)) ? expf(s[n] - m) * inv : 0.f;
 }
 
 }  // namespace stk

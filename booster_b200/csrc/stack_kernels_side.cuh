@@ -142,94 +142,142 @@ __device__ __forceinline__ float dot16(const uint4 & raw, const float * x, const
     return fmaf(__uint_as_float(raw.x), p.x, fmaf(__uint_as_float(raw.y), p.y, fmaf(__uint_as_float(raw.z), p.z, __uint_as_float(raw.w) * p.w)));
 }
 
-// Steps of few tokens: the whole end of a layer in one launch — the sum of both sub-layers, the token's own input and the norm that
-// follows. A thread-block cluster of END_CTAS blocks per token: every block forms the summed row in its shared memory, takes a share of
-// W_g's rows and writes the results into all blocks' shared memory; then a share of W_p's rows, the residual entries of that share, and
-// their part of both sums of squares, exchanged the same way. No block rewrites X before all have read it. grid (END_CTAS, T).
-constexpr int END_CTAS = 8, END_THREADS = 512;
-inline int end_slice(int E) { return ((E + END_CTAS - 1) / END_CTAS + 3) / 4 * 4; }
-inline size_t end_smem(int E, int dim) { return ((size_t) (E + 3) / 4 * 4 + (size_t) (dim + 3) / 4 * 4 + (size_t) end_slice(E)) * 4; }
+// Steps of few tokens: the end of a layer in two launches wide enough to fetch both matrices at full bandwidth. Weights are asked for
+// before anything they wait for.
+// First: every block sums the row (as k_sum_join does, but into Xs: X stays as it is while others read it) into shared memory and takes
+// SIDE_ROWS rows of W_g: G[t][i] = gelu(W_g x) e_i. grid (ceil(dim / SIDE_ROWS), T), E floats of shared memory.
+constexpr int SIDE_THREADS = 512, SIDE_ROWS = 2, SIDE_MOST = 10240;       // SIDE_MOST: the widest row these kernels take
+__device__ __forceinline__ uint4 ld_now(const void * p) {                 // stays where it is written: ahead of the waits that follow
+    uint4 v;
+    asm volatile("ld.global.nc.v4.b32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
 template <typename WT>
-__global__ void __cluster_dims__(END_CTAS, 1, 1) __launch_bounds__(END_THREADS)
-k_layer_end(const SumArgs a, const SideW s, const int32_t * __restrict__ tokens, int n_vocab, int slice, int vec_g, int vec_p, int lpr) {
-    namespace cg = cooperative_groups;
-    cg::cluster_group cluster = cg::this_cluster();
-    extern __shared__ __align__(16) float esm[];
-    __shared__ float red[32], part[2][END_CTAS];
-    constexpr int VEC = 16 / (int) sizeof(WT), NW = END_THREADS / 32;
-    const int E = a.E, dim = s.dim, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rank = (int) cluster.block_rank(), t = blockIdx.y;
-    float * xs = esm, * g = xs + (E + 3) / 4 * 4, * ys = g + (dim + 3) / 4 * 4;
-    cluster.barrier_arrive();                              // waited for before the first store into another block's shared memory
-    const int e0 = min(rank * slice, E), e1 = min(e0 + slice, E);
-    const int dper = (dim + END_CTAS - 1) / END_CTAS, d0 = min(rank * dper, dim), d1 = min(d0 + dper, dim);
-    const WT * Wg = reinterpret_cast<const WT *>(s.Wg), * Wp = reinterpret_cast<const WT *>(s.Wp);
-    {   // both shares of weights are on their way to L2 while the row is summed
-        const char * p = reinterpret_cast<const char *>(Wg + (size_t) d0 * E), * q = reinterpret_cast<const char *>(Wp + (size_t) e0 * dim);
-        const size_t np = (size_t) (d1 - d0) * E * sizeof(WT), nq = (size_t) (e1 - e0) * dim * sizeof(WT);
-        for (size_t b = (size_t) tid * 128; b < np; b += (size_t) END_THREADS * 128) asm volatile("prefetch.global.L2 [%0];" :: "l"(p + b));
-        for (size_t b = (size_t) tid * 128; b < nq; b += (size_t) END_THREADS * 128) asm volatile("prefetch.global.L2 [%0];" :: "l"(q + b));
+__global__ void __launch_bounds__(SIDE_THREADS) k_side_in(const SumArgs a, const SideW s, const int32_t * __restrict__ tokens, int n_vocab, int vec, float * __restrict__ Xs, float * __restrict__ G) {
+    extern __shared__ __align__(16) float xs[];
+    __shared__ float ps[SIDE_THREADS / 32];
+    constexpr int VEC = 16 / (int) sizeof(WT), GP = 4, WPR = SIDE_THREADS / 32 / SIDE_ROWS;      // chunks per lane asked for ahead; warps per row
+    const int E = a.E, dim = s.dim, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t = blockIdx.y;
+    const int r = blockIdx.x * SIDE_ROWS + warp / WPR, first = (warp % WPR) * 32 + lane;
+    const bool on = r < dim;
+    const WT * w = reinterpret_cast<const WT *>(s.Wg) + (size_t) (on ? r : 0) * E;
+    uint4 wg[GP];
+    if (vec) {
+#pragma unroll
+        for (int j = 0; j < GP; j++) { const int k = (j * WPR * 32 + first) * VEC; wg[j] = on && k < E ? ld_now(w + k) : make_uint4(0u, 0u, 0u, 0u); }
     }
     int tok = tokens[t];
     tok = tok < 0 ? 0 : tok >= n_vocab ? n_vocab - 1 : tok;
-    const WT * e = reinterpret_cast<const WT *>(s.table) + (size_t) tok * s.ld + s.off;
-    if ((E & 3) == 0) {
-        for (int i = tid * 4; i < E; i += END_THREADS * 4) { float v[4]; sum_chunk<4>(a, t, i, v); st_chunk<4>(xs + i, v); }
-    } else {
-        for (int i = tid; i < E; i += END_THREADS) { float v[1]; sum_chunk<1>(a, t, i, v); xs[i] = v[0]; }
-    }
+    const float e = on ? wf(reinterpret_cast<const WT *>(s.table), (size_t) tok * s.ld + s.off + r) : 0.f;
+    const auto sum = [&](int i, auto & v) {
+        constexpr int N = sizeof(v) / sizeof(float);
+        sum_chunk<N>(a, t, i, v);
+        st_chunk<N>(xs + i, v);
+        if (blockIdx.x == 0) st_chunk<N>(Xs + (size_t) t * E + i, v);
+    };
+    if ((E & 3) == 0) { for (int i = tid * 4; i < E; i += SIDE_THREADS * 4) { float v[4]; sum(i, v); } }
+    else { for (int i = tid; i < E; i += SIDE_THREADS) { float v[1]; sum(i, v); } }
     __syncthreads();
-    cluster.barrier_wait();
-    for (int r = d0 + warp; r < d1; r += NW) {             // a warp per row of W_g
-        const WT * w = Wg + (size_t) r * E;
-        const float er = wf(e, r);
-        float acc = 0.f;
-        if (vec_g) {
-#pragma unroll 8
-            for (int k = lane * VEC; k < E; k += 32 * VEC) acc += dot16(__ldg(reinterpret_cast<const uint4 *>(w + k)), xs + k, w);
-        } else {
-            for (int k = lane; k < E; k += 32) acc = fmaf(wf(w, k), xs[k], acc);
-        }
-        acc = warp_sum(acc);
-        if (lane < END_CTAS) *cluster.map_shared_rank(g + r, lane) = gelu_tanhf_(acc) * er;
+    float acc = 0.f;
+    if (vec) {
+#pragma unroll
+        for (int j = 0; j < GP; j++) { const int k = (j * WPR * 32 + first) * VEC; if (k < E) acc += dot16(wg[j], xs + k, w); }
+        for (int k = (GP * WPR * 32 + first) * VEC; k < E; k += WPR * 32 * VEC) acc += dot16(ld_now(w + k), xs + k, w);
+    } else {
+        for (int k = first; k < E; k += WPR * 32) acc = fmaf(wf(w, k), xs[k], acc);
     }
-    cluster.sync();
-    float ss = 0.f;
-    const int sub = tid % lpr, grp = tid / lpr, ngrp = END_THREADS / lpr;      // lpr lanes per row of W_p (a power of two)
-#pragma unroll 4
-    for (int base = e0; base < e1; base += ngrp) {
-        const int row = base + grp;
+    acc = warp_sum(acc);
+    if (lane == 0) ps[warp] = acc;
+    __syncthreads();
+    if (first == 0 && on) {                                // the row's warps in a fixed order
+        acc = 0.f;
+#pragma unroll
+        for (int i = 0; i < WPR; i++) acc += ps[warp + i];
+        G[(size_t) t * dim + r] = gelu_tanhf_(acc) * e;
+    }
+}
+// Second: lpr lanes (a power of two) per row of W_p, SIDE_PER rows per group of lanes: Y[t] = W_p G[t]; the block of a token that finishes
+// last (an atomic counter, no waiting) takes X[t] = Xs[t] + Y / rms(Y) wn and Hn[t] = X / rms(X) * nw, the row in registers in XV-entry
+// chunks. grid (ceil(E / rows per block), T), dim floats of shared memory.
+constexpr int SIDE_PER = 2;
+inline int side_rows_per_block(int lpr) { return SIDE_THREADS / lpr * SIDE_PER; }
+template <typename WT, int XV>
+__global__ void __launch_bounds__(SIDE_THREADS) k_side_out(const SumArgs a, const SideW s, const float * __restrict__ Xs, const float * __restrict__ G, float * __restrict__ Y, int * __restrict__ counter, int vec, int lpr) {
+    extern __shared__ __align__(16) float g[];
+    __shared__ float red[32];
+    __shared__ int last_s;
+    constexpr int VEC = 16 / (int) sizeof(WT), OWN = SIDE_MOST / (SIDE_THREADS * XV);
+    const int E = a.E, dim = s.dim, tid = threadIdx.x, t = blockIdx.y, sub = tid % lpr, grp = tid / lpr, ngrp = SIDE_THREADS / lpr, r0 = blockIdx.x * ngrp * SIDE_PER + grp;
+    const WT * Wp = reinterpret_cast<const WT *>(s.Wp);
+    uint4 wp[SIDE_PER];
+    if (vec) {
+#pragma unroll
+        for (int j = 0; j < SIDE_PER; j++) { const int r = r0 + j * ngrp; wp[j] = r < E && sub * VEC < dim ? ld_now(Wp + (size_t) r * dim + sub * VEC) : make_uint4(0u, 0u, 0u, 0u); }
+    }
+    for (int i = tid; i < dim; i += SIDE_THREADS) g[i] = G[(size_t) t * dim + i];
+    __syncthreads();
+    const size_t row = (size_t) t * E;
+#pragma unroll
+    for (int j = 0; j < SIDE_PER; j++) {
+        const int r = r0 + j * ngrp;
         float acc = 0.f;
-        if (row < e1) {
-            const WT * w = Wp + (size_t) row * dim;
-            if (vec_p) { for (int k = sub * VEC; k < dim; k += lpr * VEC) acc += dot16(__ldg(reinterpret_cast<const uint4 *>(w + k)), g + k, w); }
-            else { for (int k = sub; k < dim; k += lpr) acc = fmaf(wf(w, k), g[k], acc); }
+        if (r < E) {
+            const WT * w = Wp + (size_t) r * dim;
+            if (vec) {
+                if (sub * VEC < dim) acc = dot16(wp[j], g + sub * VEC, w);
+                for (int k = (lpr + sub) * VEC; k < dim; k += lpr * VEC) acc += dot16(ld_now(w + k), g + k, w);
+            } else {
+                for (int k = sub; k < dim; k += lpr) acc = fmaf(wf(w, k), g[k], acc);
+            }
         }
         for (int o = lpr >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-        if (sub == 0 && row < e1) { ys[row - e0] = acc; ss = fmaf(acc, acc, ss); }
+        if (sub == 0 && r < E) Y[row + r] = acc;
+    }
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) last_s = atomicAdd(counter + t, 1) == (int) gridDim.x - 1;
+    __syncthreads();
+    if (!last_s) return;
+    __threadfence();
+    if (tid == 0) counter[t] = 0;
+    float y[OWN][XV], x[OWN][XV], w[OWN][XV], f[OWN][XV], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < OWN; k++) {
+        const int i = (tid + k * SIDE_THREADS) * XV;
+        if (i < E) {
+            if constexpr (XV == 4) { const float4 v = __ldcg(reinterpret_cast<const float4 *>(Y + row + i)); y[k][0] = v.x; y[k][1] = v.y; y[k][2] = v.z; y[k][3] = v.w; }
+            else y[k][0] = __ldcg(Y + row + i);
+            ld_chunk<XV>(Xs + row + i, x[k]); ld_chunk<XV>(s.wn + i, w[k]); ld_chunk<XV>(a.nw + i, f[k]);
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < OWN; k++) if ((tid + k * SIDE_THREADS) * XV < E) {
+#pragma unroll
+        for (int e = 0; e < XV; e++) ss = fmaf(y[k][e], y[k][e], ss);
     }
     ss = block_sum(ss, red);
-    if (tid < END_CTAS) *cluster.map_shared_rank(&part[0][rank], tid) = ss;
-    cluster.sync();
-    float tot = 0.f;
-#pragma unroll
-    for (int r = 0; r < END_CTAS; r++) tot += part[0][r];  // the same order in every block
-    const float ry = 1.0f / sqrtf(tot / (float) E + a.eps);
+    const float ry = 1.0f / sqrtf(ss / (float) E + a.eps);
     ss = 0.f;
-    for (int i = e0 + tid; i < e1; i += END_THREADS) {
-        const float v = fmaf(ys[i - e0] * ry, s.wn[i], xs[i]);
-        xs[i] = v;
-        a.X[(size_t) t * E + i] = v;
-        ss = fmaf(v, v, ss);
-    }
-    if (!a.nw) return;                                     // no block reads another's shared memory any more
-    ss = block_sum(ss, red);
-    if (tid < END_CTAS) *cluster.map_shared_rank(&part[1][rank], tid) = ss;
-    cluster.sync();
-    tot = 0.f;
 #pragma unroll
-    for (int r = 0; r < END_CTAS; r++) tot += part[1][r];
-    const float rx = 1.0f / sqrtf(tot / (float) E + a.eps);
-    for (int i = e0 + tid; i < e1; i += END_THREADS) a.Hn[(size_t) t * E + i] = xs[i] * rx * a.nw[i];
+    for (int k = 0; k < OWN; k++) {
+        const int i = (tid + k * SIDE_THREADS) * XV;
+        if (i < E) {
+#pragma unroll
+            for (int e = 0; e < XV; e++) { x[k][e] = fmaf(y[k][e] * ry, w[k][e], x[k][e]); ss = fmaf(x[k][e], x[k][e], ss); }
+            st_chunk<XV>(a.X + row + i, x[k]);
+        }
+    }
+    ss = block_sum(ss, red);
+    const float rx = 1.0f / sqrtf(ss / (float) E + a.eps);
+#pragma unroll
+    for (int k = 0; k < OWN; k++) {
+        const int i = (tid + k * SIDE_THREADS) * XV;
+        if (i < E) {
+#pragma unroll
+            for (int e = 0; e < XV; e++) x[k][e] = x[k][e] * rx * f[k][e];
+            st_chunk<XV>(a.Hn + row + i, x[k]);
+        }
+    }
 }
 
 }  // namespace stk
