@@ -295,6 +295,22 @@ def test_far_keys_stand_out(tmp_path):
     p.close()
 
 
+@pytest.mark.parametrize("shape", [(1, 16, 8), (2, 64, 64), (3, 128, 128), (4, 132, 20), (5, 8, 256), (6, 256, 128), (8, 32, 128), (9, 64, 4), (17, 4, 4)], ids=str)
+def test_few_token_attention_over_many_slices(tmp_path, shape):
+    """queries per key head below, at and beyond what a block takes together, one or two 16-byte chunks per lane, several strips per warp
+    and several blocks per head: single tokens and short portions far into a sequence"""
+    R, dim, vdim = shape
+    cfg = config([att(heads=2 * R, kv_heads=2, dim=dim, vdim=vdim, rot=4, scale=1.5 / np.sqrt(dim)), att(heads=R, kv_heads=1, dim=dim, vdim=vdim, rot=4, scale=4.0 / np.sqrt(dim))], width=32, vocab=40)
+    p = Pair(tmp_path, cfg, seed=R, n_ctx=2048)
+    toks = p.tokens(700, seed=R)
+    want = p.expected(toks)
+    for cuts in ([661] + [1] * 39, [655, 7, 6, 5, 4, 3, 2, 1, 7, 7]):
+        got = p.run(toks, cuts)
+        assert err(got, want) < 2 * TOL32, cuts
+    assert err(p.run(toks[:120], [1, 2, 3, 4, 5, 6, 7]), want[:120]) < TOL32      # from the first token on
+    p.close()
+
+
 def test_steep_scores_and_angles(tmp_path):
     """peaked attention: positions one off, or another factor on the rotated entries, are far away"""
     cfg = config([att(heads=4, kv_heads=1, dim=8, rot=8, scale=3.0, mlp=dense())], width=32, vocab=40)
