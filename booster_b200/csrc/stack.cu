@@ -1176,7 +1176,9 @@ void build_bozisun(StackModel & m, const Json & cfg, const safetensors_file & sf
     if (cfg.has("embedding") && cfg.at("embedding").has("bigram")) {
         const Json & bj = cfg.at("embedding").at("bigram");
         m.pair_buckets = need_int(bj, "buckets");
-        m.pair_mul_prev = need_int(bj, "mul_prev", 0); m.pair_mul_cur = need_int(bj, "mul_cur", 0);
+        m.pair_mul_prev = bj.integer("mul_prev"); m.pair_mul_cur = bj.integer("mul_cur");
+        for (const int64_t f : { m.pair_mul_prev, m.pair_mul_cur })      // token x multiplier, twice, stays below 2^64
+            if (f < 0 || f > (int64_t) 1 << 32) throw std::runtime_error("config: bigram multipliers must lie between 0 and 2^32");
         m.pair_table = table("bigram", (int) m.pair_buckets + 1, E);
     }
     if (cfg.has("token_side")) {

@@ -3,7 +3,7 @@
 // matrix (hyper-connections), RMS norms whose weight is one number, and a soft-max attention over grouped key/value heads
 // whose options are all arguments: per-head RMS norm of queries and keys, rotation of neighbouring or half-split pairs on part
 // of a head, a cap on the scores, a logarithmic distance penalty, a sink in the denominator, values mixed with an earlier
-// layer's, a per-head output gate, and three masks (causal | chunks counted from position 0 | a sliding window with the means
+// layer's, an output gate per head or per entry, and three masks (causal | chunks counted from position 0 | a sliding window with the means
 // of whole blocks of cached keys and values standing in for what lies before the window).
 // Everything here is float32: streams, norms, positions and angles, scores and weights.
 #pragma once
@@ -583,19 +583,32 @@ __global__ void k_gqa_softmax_rows(float * __restrict__ S, int n_rows, int G, in
     const int jlo = span > 0 ? st->pos0 + (t / TQ) * TQ - span + 1 : 0;
     const int n_lo = npc + gqa_first_token(mask, p) - jlo, n_hi = npc + p - jlo, nb = gqa_blocks_seen(mask, p);     // token columns n_lo .. n_hi, block columns 0 .. nb - 1
     const float r1 = r1v ? r1v[h] : 0.f, r2 = r1v ? r2v[h] : 0.f;
+    const bool plain = !(sc.cap > 0.f) && !r1v;             // scores are products times a number: nothing to write back before the soft-max
     float mx = -INFINITY;
-    for (int n = lane; n < nb; n += 32) { const float v = gqa_score(sc, s[n], 0.f, 0.f, 0); s[n] = v; mx = fmaxf(mx, v); }
-    for (int n = n_lo + lane; n <= n_hi; n += 32) { const float v = gqa_score(sc, s[n], r1, r2, n_hi - n); s[n] = v; mx = fmaxf(mx, v); }
+    if (plain) {
+#pragma unroll 4
+        for (int n = lane; n < nb; n += 32) mx = fmaxf(mx, s[n] * sc.scale);
+#pragma unroll 8
+        for (int n = n_lo + lane; n <= n_hi; n += 32) mx = fmaxf(mx, s[n] * sc.scale);
+    } else {
+        for (int n = lane; n < nb; n += 32) { const float v = gqa_score(sc, s[n], 0.f, 0.f, 0); s[n] = v; mx = fmaxf(mx, v); }
+        for (int n = n_lo + lane; n <= n_hi; n += 32) { const float v = gqa_score(sc, s[n], r1, r2, n_hi - n); s[n] = v; mx = fmaxf(mx, v); }
+    }
     mx = warp_max(mx);
-    const float snk = sink ? sink[h] : -INFINITY;
+    const float f = plain ? sc.scale : 1.0f, snk = sink ? sink[h] : -INFINITY;
     const float m = fmaxf(mx, snk);
     float sum = 0.f;
-    for (int n = lane; n < nb; n += 32) sum += expf(s[n] - m);
-    for (int n = n_lo + lane; n <= n_hi; n += 32) sum += expf(s[n] - m);
+    for (int n = lane; n < nb; n += 32) sum += expf(s[n] * f - m);
+#pragma unroll 8
+    for (int n = n_lo + lane; n <= n_hi; n += 32) sum += expf(s[n] * f - m);
     sum = warp_sum(sum);
     const float inv = 1.0f / (sum + (sink ? expf(snk - m) : 0.f));
-    __syncwarp();                                           // the last pass walks the row from column 0: other lanes' columns
-    for (int n = lane; n < nw; n += 32) s[n] = (n < nb || (n >= n_lo && n <= n_hi)) ? expf(s[n] - m) * inv : 0.f;
+    // a lane rewrites its own columns of each range; zeros around them
+    for (int n = lane; n < nb; n += 32) s[n] = expf(s[n] * f - m) * inv;
+    for (int n = nb + lane; n < n_lo; n += 32) s[n] = 0.f;
+#pragma unroll 8
+    for (int n = n_lo + lane; n <= n_hi; n += 32) s[n] = expf(s[n] * f - m) * inv;
+    for (int n = n_hi + 1 + lane; n < nw; n += 32) s[n] = 0.f;
 }
 
 }  // namespace stk

@@ -252,7 +252,7 @@ def test_who_notices_a_changed_token(tmp_path, path):
 
 def test_pair_rows(tmp_path):
     """the first token's extra row, rows that differ in the order of a pair, multipliers whose products need more than 32 bits"""
-    for pc in ((50, 3, 7), (509, 1 << 29, (1 << 29) + 12345), (3, 0, 1), (64, 1, 0)):
+    for pc in ((50, 3, 7), (509, 1 << 29, (1 << 29) + 12345), (1021, 4294967291, 2654435761), (3, 0, 1), (64, 1, 0)):
         cfg = config([att(mlp=dense())], width=32, vocab=2000, pairs=pc, side=0)
         p = Pair(tmp_path, cfg, seed=pc[0], n_ctx=64)
         toks = p.tokens(40, seed=pc[0])
